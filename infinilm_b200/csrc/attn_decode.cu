@@ -21,6 +21,10 @@
 // Values that are the keys (use_tma 3: a cache whose V plane repeats its K plane, as the latent of a latent-attention
 // mixer does): only the K plane is copied, by a map whose box is that plane's page, and P.V reads the same tile
 // transposed. Half the bytes a page, half the shared memory a stage, so more blocks an SM.
+//
+// Two kinds of weights. Softmax, as above; or - the template's SIG - every visible key's own sigmoid of its (scaled, biased)
+// score, with no normalisation over the keys: the running maximum then stays 0, nothing is rescaled, the splits' partials are
+// plain sums and the merge adds them.
 #include <cuda.h>
 #include <cstring>
 
@@ -79,7 +83,7 @@ constexpr int AD_MERGE_ROUND = 16;
 
 template <int WPR>
 __device__ __forceinline__ void ad_merge_row(float* fs, float* comb, const float* o_part, const float* ml_part, size_t row, int n_valid,
-                                             int n_splits, __nv_bfloat16* __restrict__ out, int lane, int sub, float sink_log2) {
+                                             int n_splits, __nv_bfloat16* __restrict__ out, int lane, int sub, float sink_log2, int plain_sum) {
     const size_t pr0 = row * n_splits;
     const int d_first = lane * 4;
     float4 v[AD_MERGE_ROUND];
@@ -111,7 +115,7 @@ __device__ __forceinline__ void ad_merge_row(float* fs, float* comb, const float
     L = il_warp_sum(L);
     __syncwarp();
     L += exp2f(sink_log2 - M);                    // the sink: one more key without a value (-inf: none, adds 0)
-    const float inv = 1.f / L;
+    const float inv = plain_sum ? 1.f : 1.f / L;  // (weights that are no softmax: every maximum is 0, every factor 1)
     for (int d = d_first; d < AT_HD; d += 128) {
         float4 acc = zero4;
         for (int i0 = 0; sub + WPR * i0 < n_valid; i0 += AD_MERGE_ROUND) {
@@ -160,6 +164,7 @@ __device__ __forceinline__ void ad_merge_row(float* fs, float* comb, const float
 // (qkv, and o_part / ml_part in the merge, are written by the kernel before and read after a wait that is not the
 // kernel's first statement: they are not declared __restrict__, so that no load of them is treated as read-only
 // data and scheduled above the wait.)
+template <bool SIG>
 __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_kernel(
     const __nv_bfloat16* qkv, int row_stride, const __nv_bfloat16* __restrict__ cache,
     const int* __restrict__ block_table, int bt_stride, const int* __restrict__ entry_kvlen, int nh, int nkv,
@@ -208,7 +213,7 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_kernel(
     for (int i = 0; i < AT_NT; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    float m[2] = {SIG ? 0.f : -INFINITY, SIG ? 0.f : -INFINITY}, l[2] = {0.f, 0.f};
 
     const int n_my = (p1 - p0 - warp + AD_WARPS - 1) / AD_WARPS;   // pages p0+warp, +4, ...
     // Page ids of this warp's iterations, 32 at a time: lane l holds the id of iteration base + l, so the
@@ -304,8 +309,17 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_kernel(
                 const int key = key0 + nt * 8 + (j & 1);
                 float v = s[nt][j] * scale_log2;
                 if (dist_bias) v += db_near ? db_row[j >> 1][max(0, min(kvlen - 1 - key, dist_far)) * nh] * 1.4426950408889634f : db_far[j >> 1];
-                s[nt][j] = (key >= lo && key < hi) ? v : -INFINITY;
+                if (SIG) s[nt][j] = (key >= lo && key < hi) ? il_sigmoid_log2_fast(v) : 0.f;
+                else s[nt][j] = (key >= lo && key < hi) ? v : -INFINITY;
             }
+        if (SIG) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                pf[h] = at_pack_bf16(s[0][2 * h], s[0][2 * h + 1]);
+                pf[2 + h] = at_pack_bf16(s[1][2 * h], s[1][2 * h + 1]);
+            }
+            return;
+        }
 #pragma unroll
         for (int h = 0; h < 2; ++h) {             // h = 0: row lane/4, h = 1: row lane/4 + 8
             float mx = fmaxf(fmaxf(s[0][2 * h], s[0][2 * h + 1]), fmaxf(s[1][2 * h], s[1][2 * h + 1]));
@@ -456,7 +470,7 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_kernel(
                 L += ((mw == -INFINITY) ? 0.f : exp2f(mw - M)) * sm_ml[(w * 16 + r) * 2 + 1];
             }
             if (sink) L += exp2f(sink[head0 + r] * 1.4426950408889634f - M);      // as the merge adds it
-            const float inv = 1.f / L;
+            const float inv = SIG ? 1.f : 1.f / L;
             const uint32_t a = at_pack_bf16(acc.x * inv, acc.y * inv), b = at_pack_bf16(acc.z * inv, acc.w * inv);
             *reinterpret_cast<uint2*>(out_direct + pr * AT_HD + d) = make_uint2(a, b);
             continue;
@@ -482,7 +496,7 @@ template <int WPR>
 __global__ void __launch_bounds__(128) attn_decode_merge_kernel(const float* o_part, const float* ml_part,
                                                                 const int* __restrict__ entry_kvlen, int nh, int n_rows, int window,
                                                                 int pages_per_split, int n_splits, __nv_bfloat16* __restrict__ out,
-                                                                const float* __restrict__ sink) {
+                                                                const float* __restrict__ sink, int plain_sum) {
     __shared__ float fs[4][AD_MAX_SPLITS];
     __shared__ __align__(16) float comb[WPR > 1 ? WPR * AT_HD : 4];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -502,7 +516,7 @@ __global__ void __launch_bounds__(128) attn_decode_merge_kernel(const float* o_p
             for (int d = lane * 4; d < AT_HD; d += 128) *reinterpret_cast<uint2*>(out + (size_t)row * AT_HD + d) = make_uint2(0u, 0u);
         return;
     }
-    ad_merge_row<WPR>(fs[warp], comb, o_part, ml_part, (size_t)row, n_valid, n_splits, out, lane, warp % WPR, sink_log2);
+    ad_merge_row<WPR>(fs[warp], comb, o_part, ml_part, (size_t)row, n_valid, n_splits, out, lane, warp % WPR, sink_log2, plain_sum);
 }
 
 // Launches the attention kernel and, for more than one split, the merge. Scratch: o_part float32 [n_decode*nh*n_splits*head_dim], ml_part [n_decode*nh*n_splits*2].
@@ -510,7 +524,7 @@ static int ad_launch(const void* qkv, int row_stride, void* out, const void* cac
                      const int* entry_kvlen, int n_decode, int nh, int nkv, float scale, int window, int pages_per_split,
                      int n_splits, float* o_part, float* ml_part, cudaStream_t stream, const CUtensorMap* kv_map = nullptr,
                      int* status = nullptr, const float* sink = nullptr, int v_is_k = 0, const float* dist_bias = nullptr,
-                     int dist_far = 0) {
+                     int dist_far = 0, int sigmoid = 0) {
     static CUtensorMap no_map;                    // passed when there is no map: the kernel does not look at it
     int use_tma = (AD_TMA_OK && kv_map && status) ? 1 : 0;
     auto filled = [&](int i) {                    // maps behind the first are all zero where the driver did not take them
@@ -527,16 +541,20 @@ static int ad_launch(const void* qkv, int row_stride, void* out, const void* cac
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev >= 0 && dev < 64 && !attr_set[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_decode_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM);
         if (e != cudaSuccess) return 1000 + (int)e;
         attr_set[dev] = true;
     }
     const int G = nh / nkv, row_tiles = (G + 15) / 16;
     dim3 grid(n_splits, nkv * row_tiles, n_decode);
-    IL_LAUNCH(attn_decode_kernel, grid, AD_WARPS * 32, smem_bytes, stream,
-        (const __nv_bfloat16*)qkv, row_stride, (const __nv_bfloat16*)cache, block_table, bt_stride, entry_kvlen, nh, nkv,
-        scale * 1.4426950408889634f, window, pages_per_split, n_splits, o_part, ml_part, use_tma ? *kv_map : no_map, page_map, use_tma, status,
-        n_splits == 1 ? (__nv_bfloat16*)out : (__nv_bfloat16*)nullptr, sink, dist_bias, dist_far);
+#define AD_GO(SIG)                                                                                                                           \
+    IL_LAUNCH(attn_decode_kernel<SIG>, grid, AD_WARPS * 32, smem_bytes, stream, (const __nv_bfloat16*)qkv, row_stride,                       \
+              (const __nv_bfloat16*)cache, block_table, bt_stride, entry_kvlen, nh, nkv, scale * 1.4426950408889634f, window, pages_per_split, \
+              n_splits, o_part, ml_part, use_tma ? *kv_map : no_map, page_map, use_tma, status,                                              \
+              n_splits == 1 ? (__nv_bfloat16*)out : (__nv_bfloat16*)nullptr, sink, dist_bias, dist_far)
+    if (sigmoid) AD_GO(true); else AD_GO(false);
+#undef AD_GO
     if (n_splits == 1) {                          // every row is final as the attention kernel leaves it: no merge
         IL_LAUNCH_CHECK();
         return IL_OK;
@@ -544,10 +562,10 @@ static int ad_launch(const void* qkv, int row_stride, void* out, const void* cac
     const int n_rows = n_decode * nh;
     if (n_splits > AD_MERGE_WIDE_FROM) {
         IL_LAUNCH(attn_decode_merge_kernel<4>, n_rows, 128, 0, stream, (const float*)o_part, (const float*)ml_part, entry_kvlen, nh, n_rows, window,
-                  pages_per_split, n_splits, (__nv_bfloat16*)out, sink);
+                  pages_per_split, n_splits, (__nv_bfloat16*)out, sink, sigmoid);
     } else {
         IL_LAUNCH(attn_decode_merge_kernel<1>, (n_rows + 3) / 4, 128, 0, stream, (const float*)o_part, (const float*)ml_part, entry_kvlen, nh, n_rows,
-                  window, pages_per_split, n_splits, (__nv_bfloat16*)out, sink);
+                  window, pages_per_split, n_splits, (__nv_bfloat16*)out, sink, sigmoid);
     }
     IL_LAUNCH_CHECK();
     return IL_OK;
@@ -562,8 +580,8 @@ static int ad_resident_blocks(int v_is_k) {
     const int k = (v_is_k && AD_TMA_OK) ? 1 : 0, smem = k ? AD_SMEM_K : AD_SMEM;
     if (cached[k][dev]) return cached[k][dev];
     int per_sm = 0, sms = 0;
-    if (cudaFuncSetAttribute(attn_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM) != cudaSuccess ||
-        cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attn_decode_kernel, AD_WARPS * 32, smem) != cudaSuccess ||
+    if (cudaFuncSetAttribute(attn_decode_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM) != cudaSuccess ||
+        cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attn_decode_kernel<false>, AD_WARPS * 32, smem) != cudaSuccess ||
         cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) {
         cudaGetLastError();
         return 0;
@@ -581,14 +599,15 @@ IL_EXPORT int il_attn_decode(const void* qkv, int row_stride, void* out, const v
                              int bt_stride, const int* entry_kvlen, int page_size, int n_decode, int nh, int nkv, int hd,
                              float scale, int window, int pages_per_split, int n_splits, float* o_part, float* ml_part,
                              const void* kv_map, int* status, const float* sink, int v_is_k, const float* dist_bias, int dist_far,
-                             cudaStream_t stream) {
+                             int sigmoid, cudaStream_t stream) {
     if (n_decode <= 0) return IL_OK;
+    if (sigmoid && sink) return IL_BAD_ARG;       // a sink is a term of a softmax's denominator
     if (dist_bias && (dist_far < 0 || (long long)(dist_far + 1) * nh > 0x7fffffffLL)) return IL_BAD_ARG;
     if (hd != HEAD_DIM || page_size != AD_PAGE) return IL_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || pages_per_split < 0 || n_splits <= 0) return IL_BAD_ARG;
     if (n_splits > AD_MAX_SPLITS) return IL_UNSUPPORTED;
     return ad_launch(qkv, row_stride, out, cache, block_table, bt_stride, entry_kvlen, n_decode, nh, nkv, scale, window,
-                     pages_per_split, n_splits, o_part, ml_part, stream, (const CUtensorMap*)kv_map, status, sink, v_is_k, dist_bias, dist_far);
+                     pages_per_split, n_splits, o_part, ml_part, stream, (const CUtensorMap*)kv_map, status, sink, v_is_k, dist_bias, dist_far, sigmoid);
 }
 
 // Writes four tensor maps (4 x 128 bytes at `out_maps`) of one layer's cache, [pages][2][kv heads][16][head_dim] bfloat16:

@@ -8,6 +8,8 @@
 //   O += P.V with P rounded to bfloat16. Pages wholly above a warp's last query position, or
 //   wholly behind its window, are skipped by that warp.
 //
+//   SIG: no softmax - a visible key's weight is the sigmoid of its (scaled, biased) score, not normalised over the keys.
+//
 //   grid (tiles, kv heads). Tiles are numbered over the entries [first_entry, n_entries) in
 //   order; a block finds its entry by walking entry_qstart.
 #include "attn_mma.cuh"
@@ -28,6 +30,7 @@ __device__ __forceinline__ float ap_ex2(float x) {
     return y;
 }
 
+template <bool SIG>
 __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
     const __nv_bfloat16* __restrict__ qkv, int row_stride, __nv_bfloat16* __restrict__ out,
     const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_table, int bt_stride,
@@ -192,7 +195,7 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
         }
         float corr[2], msafe[2];
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
+        for (int h = 0; h < 2 && !SIG; ++h) {
             mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
             mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
             const float mn = fmaxf(m[h], mx[h] * scale_log2);      // running maximum of the scaled scores (scale > 0)
@@ -200,7 +203,7 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
             msafe[h] = (mn == -INFINITY) ? 0.f : mn;
             m[h] = mn;
         }
-        if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {   // nothing to rescale once the maxima have settled
+        if (!SIG && __any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {   // nothing to rescale once the maxima have settled
 #pragma unroll
             for (int nt = 0; nt < AT_NT; ++nt) {
                 o[nt][0] *= corr[0];
@@ -216,6 +219,11 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
             uint32_t pf[4];
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
+                if (SIG) {
+                    pf[h] = at_pack_bf16(il_sigmoid_log2_fast(s[p][0][2 * h] * scale_log2), il_sigmoid_log2_fast(s[p][0][2 * h + 1] * scale_log2));
+                    pf[2 + h] = at_pack_bf16(il_sigmoid_log2_fast(s[p][1][2 * h] * scale_log2), il_sigmoid_log2_fast(s[p][1][2 * h + 1] * scale_log2));
+                    continue;
+                }
                 // 2^(s * scale - m) with one fused multiply-add per score
                 const float a = ap_ex2(fmaf(s[p][0][2 * h], scale_log2, -msafe[h])), b = ap_ex2(fmaf(s[p][0][2 * h + 1], scale_log2, -msafe[h]));
                 const float c = ap_ex2(fmaf(s[p][1][2 * h], scale_log2, -msafe[h])), d = ap_ex2(fmaf(s[p][1][2 * h + 1], scale_log2, -msafe[h]));
@@ -226,7 +234,7 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
             at_pv_16keys(o, pf, st + p * AP_PAGE_BYTES + AP_PAGE * AT_ROW_BYTES, lane);
         }
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
+        for (int h = 0; h < 2 && !SIG; ++h) {
             rs[h] += __shfl_xor_sync(0xffffffffu, rs[h], 1);
             rs[h] += __shfl_xor_sync(0xffffffffu, rs[h], 2);
             l[h] = l[h] * corr[h] + rs[h];
@@ -238,7 +246,7 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
     for (int h = 0; h < 2; ++h) {
         if (!rvalid[h]) continue;
         // a sink joins the denominator as one more key without a value: 2^(sink * log2(e) - m), its score not scaled
-        const float inv = 1.f / (sink ? l[h] + ap_ex2(fmaf(sink[rhead[h]], 1.4426950408889634f, -m[h])) : l[h]);
+        const float inv = SIG ? 1.f : 1.f / (sink ? l[h] + ap_ex2(fmaf(sink[rhead[h]], 1.4426950408889634f, -m[h])) : l[h]);
         __nv_bfloat16* orow = optr[h];
 #pragma unroll
         for (int nt = 0; nt < AT_NT; ++nt) {
@@ -252,21 +260,23 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
 IL_EXPORT int il_attn_prefill(const void* qkv, int row_stride, void* out, const void* cache, const int* block_table,
                               int bt_stride, const int* entry_qstart, const int* entry_kvlen, int page_size,
                               int first_entry, int n_entries, int n_tiles_total, int nh, int nkv, int hd, float scale,
-                              int window, const float* sink, const float* dist_bias, int dist_far, cudaStream_t stream) {
+                              int window, const float* sink, const float* dist_bias, int dist_far, int sigmoid, cudaStream_t stream) {
     if (n_tiles_total <= 0 || first_entry >= n_entries) return IL_OK;
     if (dist_bias && (dist_far < 0 || !(scale > 0.f) || (long long)(dist_far + 1) * nh > 0x7fffffffLL)) return IL_BAD_ARG;
+    if (sigmoid && (sink || !(scale > 0.f))) return IL_BAD_ARG;      // (a masked score is -inf before it is scaled)
     if (hd != HEAD_DIM || page_size != AP_PAGE) return IL_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) return IL_BAD_ARG;
     const int G = nh / nkv;
     if (G > AP_ROWS) return IL_UNSUPPORTED;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, AP_SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AP_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AP_SMEM);
         if (e != cudaSuccess) return 1000 + (int)e;
         attr_set = true;
     }
     dim3 grid(n_tiles_total, nkv);
-    attn_prefill_kernel<<<grid, AP_WARPS * 32, AP_SMEM, stream>>>(
+    (sigmoid ? attn_prefill_kernel<true> : attn_prefill_kernel<false>)<<<grid, AP_WARPS * 32, AP_SMEM, stream>>>(
         (const __nv_bfloat16*)qkv, row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)cache, block_table, bt_stride,
         entry_qstart, entry_kvlen, first_entry, n_entries, nh, nkv, scale * 1.4426950408889634f, window, AP_ROWS / G, sink, dist_bias, dist_far,
         1.f / scale);

@@ -29,6 +29,10 @@
 //   busy 1,000 clocks a tile. Two softmax threads a row (71 against 53 us), one block per SM with two tiles of 128
 //   rows (67 us) and tiles of 128 keys with single-buffered scores (no gain) were slower or equal.
 //
+//   SIG: no softmax - a visible key's weight is the sigmoid of its (scaled, biased) score, not normalised over the keys. No
+//   maximum, no rescaling of O, no row sums; a score costs an exponential and half a reciprocal (two scores share one:
+//   1/a = b/(ab)), so the special-function unit is the busier half of a tile.
+//
 //   Pages past the entry's last page are read as the last page again (finite values the mask removes).
 //   Every mbarrier wait is bounded; one that runs out sets *status and all roles leave their loops.
 //
@@ -83,6 +87,7 @@ __device__ __forceinline__ uint32_t pt_pack(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
+template <bool SIG>
 __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5_kernel(
     const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* __restrict__ qkv, int row_stride,
     __nv_bfloat16* __restrict__ out, const int* __restrict__ block_table, int bt_stride, const int* __restrict__ entry_qstart,
@@ -313,31 +318,45 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
                     if (!(key <= rpos && key >= rlo)) sv[c] = __float_as_uint(-INFINITY);
                 }
             }
-            float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains: a single one is all latency
+            bool raise = false;
+            float corr = 1.f;
+            if constexpr (SIG) {
+                // 1 / (1 + 2^-v): the exponent is kept below 60 so that the product of two denominators stays finite, and a key
+                // that the mask took out (-inf) is set to zero
 #pragma unroll
-            for (int c = 0; c < PT_KEYS; c += 4)
+                for (int c = 0; c < PT_KEYS; c += 2) {
+                    const float s0 = __uint_as_float(sv[c]), s1 = __uint_as_float(sv[c + 1]);
+                    const float a = 1.f + pt_ex2(fminf(s0 * -scale_log2, 60.f)), bb = 1.f + pt_ex2(fminf(s1 * -scale_log2, 60.f));
+                    const float rr = __fdividef(1.f, a * bb);
+                    sv[c >> 1] = pt_pack(s0 == -INFINITY ? 0.f : rr * bb, s1 == -INFINITY ? 0.f : rr * a);
+                }
+            } else {
+                float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains: a single one is all latency
 #pragma unroll
-                for (int i = 0; i < 4; ++i) mx4[i] = fmaxf(mx4[i], __uint_as_float(sv[c + i]));
-            const float mxs = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;      // scale > 0
-            const bool raise = mxs > m + PT_RAISE;            // also the first keys a row sees (m = -inf)
-            const float m_new = raise ? mxs : m;
-            const float corr = raise ? pt_ex2(m - m_new) : 1.f;   // 0 when nothing was summed yet
-            const float msafe = (m_new == -INFINITY) ? 0.f : m_new;
-            float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+                for (int c = 0; c < PT_KEYS; c += 4)
 #pragma unroll
-            for (int c = 0; c < PT_KEYS; c += 2) {
-                const float a = pt_ex2(fmaf(__uint_as_float(sv[c]), scale_log2, -msafe));
-                const float bb = pt_ex2(fmaf(__uint_as_float(sv[c + 1]), scale_log2, -msafe));
-                sum4[(c >> 1) & 3] += a + bb;
-                sv[c >> 1] = pt_pack(a, bb);
+                    for (int i = 0; i < 4; ++i) mx4[i] = fmaxf(mx4[i], __uint_as_float(sv[c + i]));
+                const float mxs = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;      // scale > 0
+                raise = mxs > m + PT_RAISE;                  // also the first keys a row sees (m = -inf)
+                const float m_new = raise ? mxs : m;
+                corr = raise ? pt_ex2(m - m_new) : 1.f;   // 0 when nothing was summed yet
+                const float msafe = (m_new == -INFINITY) ? 0.f : m_new;
+                float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int c = 0; c < PT_KEYS; c += 2) {
+                    const float a = pt_ex2(fmaf(__uint_as_float(sv[c]), scale_log2, -msafe));
+                    const float bb = pt_ex2(fmaf(__uint_as_float(sv[c + 1]), scale_log2, -msafe));
+                    sum4[(c >> 1) & 3] += a + bb;
+                    sv[c >> 1] = pt_pack(a, bb);
+                }
+                l = l * corr + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
+                m = m_new;
             }
-            l = l * corr + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
-            m = m_new;
             if (j > 0) {
                 // P's place in shared memory is free, and O holds the tiles before this one, only when their last product is through
                 if (!t5_mbar_wait(o_done, (uint32_t)(j - 1) & 1u, PT_SPIN)) { atomicExch(status, 37); ok = false; break; }
                 t5_fence_after();
-                if (__any_sync(0xffffffffu, raise)) {
+                if (!SIG && __any_sync(0xffffffffu, raise)) {
 #pragma unroll
                     for (int c0 = 0; c0 < PT_HD; c0 += 32) {
                         uint32_t ov[32];
@@ -366,7 +385,7 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
                 t5_fence_after();
                 // a sink joins the denominator as one more key without a value: 2^(sink * log2(e) - m), its score not scaled
                 if (sink && rvalid) l += pt_ex2(fmaf(sink[g * G + hh], 1.4426950408889634f, -m));
-                const float inv = (l > 0.f) ? 1.f / l : 0.f;
+                const float inv = SIG ? 1.f : (l > 0.f) ? 1.f / l : 0.f;
                 // The rows go out through shared memory (Q's place: every product that reads Q is through): a thread owns a
                 // row of tensor memory, but 16-byte stores 8 KB apart cost a block 2 us; a warp's 32 rows are stored
                 // 32 / CH at a time instead, CH lanes a row, each row's bytes contiguous.
@@ -418,9 +437,10 @@ IL_EXPORT int il_attn_prefill_tc5_rows() { return PT_ROWS; }
 IL_EXPORT int il_attn_prefill_tc5(const void* qkv, int row_stride, void* out, const void* kv_map, const int* block_table,
                                   int bt_stride, const int* entry_qstart, const int* entry_kvlen, int page_size, int first_entry,
                                   int n_entries, int n_tiles_total, int nh, int nkv, int hd, float scale, int window, int* status,
-                                  const float* sink, const float* dist_bias, int dist_far, cudaStream_t stream) {
+                                  const float* sink, const float* dist_bias, int dist_far, int sigmoid, cudaStream_t stream) {
     if (n_tiles_total <= 0 || first_entry >= n_entries) return IL_OK;
     if (dist_bias && (dist_far < 0 || (long long)(dist_far + 1) * nh > 0x7fffffffLL)) return IL_BAD_ARG;
+    if (sigmoid && sink) return IL_BAD_ARG;       // a sink is a term of a softmax's denominator
     if (hd != HEAD_DIM || page_size != PT_PAGE || !kv_map || !status) return IL_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) return IL_BAD_ARG;
     const int G = nh / nkv;
@@ -430,16 +450,18 @@ IL_EXPORT int il_attn_prefill_tc5(const void* qkv, int row_stride, void* out, co
     cudaGetDevice(&dev);
     static bool attr_set[64];
     if (dev >= 0 && dev < 64 && !attr_set[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc5_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, PT_SMEM);
-        if (e == cudaSuccess)
-            e = cudaFuncSetAttribute(attn_prefill_tc5_kernel, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+        cudaError_t e = cudaSuccess;
+        for (auto k : {attn_prefill_tc5_kernel<false>, attn_prefill_tc5_kernel<true>}) {
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, PT_SMEM);
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+        }
         if (e != cudaSuccess) return 1000 + (int)e;
         attr_set[dev] = true;
     }
     CUtensorMap map;
     memcpy(&map, kv_map, sizeof(map));
     dim3 grid(n_tiles_total, nkv);
-    attn_prefill_tc5_kernel<<<grid, PT_THREADS, PT_SMEM, stream>>>(
+    (sigmoid ? attn_prefill_tc5_kernel<true> : attn_prefill_tc5_kernel<false>)<<<grid, PT_THREADS, PT_SMEM, stream>>>(
         map, (const __nv_bfloat16*)qkv, row_stride, (__nv_bfloat16*)out, block_table, bt_stride, entry_qstart, entry_kvlen,
         first_entry, n_entries, nh, nkv, scale * 1.4426950408889634f, window, PT_ROWS / G, status, sink, dist_bias, dist_far, 1.f / scale);
     IL_LAUNCH_CHECK();

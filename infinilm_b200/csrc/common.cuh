@@ -92,8 +92,28 @@ __device__ __forceinline__ float il_gelu_tanh_mul(float g, float u) {
     const float a = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     return 0.5f * g * (1.f + tanhf(a)) * u;
 }
-// The gate of a gated feed-forward by number: 1 SiLU, 2 the tanh form of GELU.
-enum { IL_ACT_SILU = 1, IL_ACT_GELU_TANH = 2 };
+// A clamped gate: g' = min(g, limit), u' = u kept within -limit .. limit, result g' * sigmoid(alpha g') * (u' + 1).
+__device__ __forceinline__ float il_clamped_glu_fast(float g, float u, float limit, float alpha) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return __fmul_rn(__fdividef(g, __fadd_rn(1.f, __expf(__fmul_rn(-alpha, g)))), __fadd_rn(u, 1.f));
+}
+__device__ __forceinline__ float il_clamped_glu(float g, float u, float limit, float alpha) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+}
+// The gate of a gated feed-forward by number: 1 SiLU, 2 the tanh form of GELU, 3 the clamped gate (which has two numbers
+// of its own, limit and alpha).
+enum { IL_ACT_SILU = 1, IL_ACT_GELU_TANH = 2, IL_ACT_CLAMPED = 3 };
+
+// 1 / (1 + 2^-v), the logistic function of v / log2(e): -inf gives 0. Exponential and reciprocal by the fast units (relative
+// error near 2^-21).
+__device__ __forceinline__ float il_sigmoid_log2_fast(float v) {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(-v));
+    return __fdividef(1.f, 1.f + fminf(e, 1e38f));
+}
 
 // ---- programmatic dependent launch --------------------------------------------------------------
 // Kernels of the decode path are launched so that the next kernel in the stream may become resident

@@ -5,7 +5,8 @@
 //   batched: every group has all M rows, and group g reads A, W and writes C at a fixed element offset g * stride
 //            (one product per head over column ranges of shared rows).
 // Epilogues: plain; GLU - W_g holds N gate rows and then N up rows, C = silu(gate) * up; gated - C is multiplied by
-// sigmoid(G[m, g * gate_gs + n]). Products accumulate in f32 in the order of K whatever the tile, one accumulator per
+// sigmoid(G[m, g * gate_gs + n * gate_ns]) (gate_ns 0: one gate per group). `row_scale` multiplies a row's products before the
+// epilogue: a factor per row of A, or - scale_by_place - per place of the sorted order. Products accumulate in f32 in the order of K whatever the tile, one accumulator per
 // output element, so a row's result does not depend on what else is in the batch. float32 runs on the FP32 pipes
 // (FFMA); bfloat16 runs on the tensor cores (mma.sync m16n8k16, operands staged by cp.async in a three-stage ring: a
 // block streams a tile of 64 weight rows over all of K once, against up to 32 rows of its group, which is what a decode
@@ -35,7 +36,8 @@ __global__ void __launch_bounds__(128) gemm_grouped_mma_kernel(const __nv_bfloat
                                                                const __nv_bfloat16* __restrict__ W, int ldw, long long w_gs,
                                                                __nv_bfloat16* __restrict__ C, int ldc, long long c_gs,
                                                                const int* __restrict__ group_off, int n_groups, int M, int N, int K,
-                                                               const __nv_bfloat16* gate, int ld_gate, long long gate_gs, const float* row_scale) {
+                                                               const __nv_bfloat16* gate, int ld_gate, long long gate_gs, int gate_ns, const float* row_scale,
+                                                               int scale_by_place) {
     using namespace ggm;
     constexpr int MT = BM / 16, NW = GLU ? 2 : 1;
     constexpr int A_BYTES = BM * ROW, W_BYTES = BN * ROW, STAGE_BYTES = A_BYTES + NW * W_BYTES;
@@ -150,7 +152,7 @@ __global__ void __launch_bounds__(128) gemm_grouped_mma_kernel(const __nv_bfloat
             const int p = r0 + mt * 16 + (lane >> 2) + 8 * h;
             if (p >= r1) continue;
             // a factor per source row (the rstd of a norm that the rows of A have not been divided by yet)
-            const float rs = row_scale ? row_scale[a_rows ? a_rows[p] : p] : 1.f;
+            const float rs = row_scale ? row_scale[a_rows && !scale_by_place ? a_rows[p] : p] : 1.f;
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt) {
                 float out2[2];
@@ -165,7 +167,7 @@ __global__ void __launch_bounds__(128) gemm_grouped_mma_kernel(const __nv_bfloat
                             v = gt / (1.f + expf(-gt)) * up;
                         }
                         if (gate) {
-                            const float gt = __bfloat162float(gate[(size_t)p * ld_gate + (size_t)g * gate_gs + gn]);
+                            const float gt = __bfloat162float(gate[(size_t)p * ld_gate + (size_t)g * gate_gs + (size_t)gn * gate_ns]);
                             v = __bfloat162float(__float2bfloat16_rn(v)) / (1.f + expf(-gt));
                         }
                     }
@@ -186,7 +188,8 @@ template <typename TA, bool GLU>
 __global__ void __launch_bounds__(256) gemm_grouped_kernel(const TA* A, int lda, long long a_gs, const int* __restrict__ a_rows,
                                                            const TA* __restrict__ W, int ldw, long long w_gs, TA* __restrict__ C, int ldc,
                                                            long long c_gs, const int* __restrict__ group_off, int n_groups, int M, int N,
-                                                           int K, const TA* gate, int ld_gate, long long gate_gs) {
+                                                           int K, const TA* gate, int ld_gate, long long gate_gs, int gate_ns, const float* row_scale,
+                                                           int scale_by_place) {
     constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[GLU ? 2 : 1][BK][BN + 4];
@@ -267,18 +270,19 @@ __global__ void __launch_bounds__(256) gemm_grouped_kernel(const TA* A, int lda,
     for (int i = 0; i < TM; ++i) {
         const int p = r0 + ty * TM + i;
         if (p >= r1) continue;
+        const float rs = row_scale ? row_scale[a_rows && !scale_by_place ? a_rows[p] : p] : 1.f;
 #pragma unroll
         for (int j = 0; j < TN; ++j) {
             const int gn = n0 + tx * TN + j;
             if (gn >= N) continue;
-            float v = acc[i][j];
+            float v = acc[i][j] * rs;
             if (GLU) {
                 // the gate and up products are rounded to the activation type first, as two separate products would be
-                const float gt = il_to_f(il_from_f<TA>(v)), up = il_to_f(il_from_f<TA>(acc2[i][j]));
+                const float gt = il_to_f(il_from_f<TA>(v)), up = il_to_f(il_from_f<TA>(acc2[i][j] * rs));
                 v = gt / (1.f + expf(-gt)) * up;
             }
             if (gate) {
-                const float gt = il_to_f(gate[(size_t)p * ld_gate + (size_t)g * gate_gs + gn]);
+                const float gt = il_to_f(gate[(size_t)p * ld_gate + (size_t)g * gate_gs + (size_t)gn * gate_ns]);
                 v = il_to_f(il_from_f<TA>(v)) / (1.f + expf(-gt));
             }
             Cg[(size_t)p * ldc + gn] = il_from_f<TA>(v);
@@ -292,7 +296,7 @@ IL_EXPORT int il_gemm_grouped_max_tiles(int M, int n_groups) { return (M + 63) /
 template <int BM, bool GLU>
 static int launch_mma(const void* A, int lda, long long a_gs, const int* a_rows, const void* W, int ldw, long long w_gs, void* C, int ldc,
                       long long c_gs, const int* group_off, int n_groups, int M, int N, int K, const void* gate, int ld_gate, long long gate_gs,
-                      const float* row_scale, cudaStream_t stream) {
+                      int gate_ns, const float* row_scale, int scale_by_place, cudaStream_t stream) {
     constexpr int smem = ggm::smem_bytes<BM, GLU>();
     static bool attr_set[64];
     int dev = 0;
@@ -305,14 +309,15 @@ static int launch_mma(const void* A, int lda, long long a_gs, const int* a_rows,
     dim3 grid((N + ggm::BN - 1) / ggm::BN, group_off ? (M + BM - 1) / BM + n_groups : (M + BM - 1) / BM, group_off ? 1 : n_groups);
     if (grid.y > 65535 || grid.z > 65535) return IL_UNSUPPORTED;
     IL_LAUNCH((gemm_grouped_mma_kernel<BM, GLU>), grid, 128, smem, stream, (const __nv_bfloat16*)A, lda, a_gs, a_rows, (const __nv_bfloat16*)W, ldw,
-              w_gs, (__nv_bfloat16*)C, ldc, c_gs, group_off, n_groups, M, N, K, (const __nv_bfloat16*)gate, ld_gate, gate_gs, row_scale);
+              w_gs, (__nv_bfloat16*)C, ldc, c_gs, group_off, n_groups, M, N, K, (const __nv_bfloat16*)gate, ld_gate, gate_gs, gate_ns, row_scale, scale_by_place);
     IL_LAUNCH_CHECK();
     return IL_OK;
 }
 
 IL_EXPORT int il_gemm_grouped(const void* A, int act_kind, int lda, long long a_gs, const int* a_rows, const void* W, int ldw, long long w_gs,
                               void* C, int ldc, long long c_gs, const int* group_off, int n_groups, int M, int N, int K, int glu,
-                              const void* gate, int ld_gate, long long gate_gs, const float* row_scale, cudaStream_t stream) {
+                              const void* gate, int ld_gate, long long gate_gs, int gate_ns, const float* row_scale, int scale_by_place,
+                              cudaStream_t stream) {
     if (M <= 0 || N <= 0 || n_groups <= 0) return IL_OK;
     if (K <= 0 || (glu && gate)) return IL_BAD_ARG;
     if (act_kind == IL_BF16 && K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0 && a_gs % 8 == 0 && w_gs % 8 == 0 && !((uintptr_t)A & 15) &&
@@ -320,17 +325,16 @@ IL_EXPORT int il_gemm_grouped(const void* A, int act_kind, int lda, long long a_
         // rows of 16-byte chunks: the tensor-core kernel. Few rows a group (a decode step): tiles of 32 rows; else 64.
         const bool few = group_off ? M <= 32 * n_groups : M <= 32;
         if (glu)
-            return few ? launch_mma<32, true>(A, lda, a_gs, a_rows, W, ldw, w_gs, C, ldc, c_gs, group_off, n_groups, M, N, K, gate, ld_gate, gate_gs, row_scale, stream)
-                       : launch_mma<64, true>(A, lda, a_gs, a_rows, W, ldw, w_gs, C, ldc, c_gs, group_off, n_groups, M, N, K, gate, ld_gate, gate_gs, row_scale, stream);
-        return few ? launch_mma<32, false>(A, lda, a_gs, a_rows, W, ldw, w_gs, C, ldc, c_gs, group_off, n_groups, M, N, K, gate, ld_gate, gate_gs, row_scale, stream)
-                   : launch_mma<64, false>(A, lda, a_gs, a_rows, W, ldw, w_gs, C, ldc, c_gs, group_off, n_groups, M, N, K, gate, ld_gate, gate_gs, row_scale, stream);
+            return few ? launch_mma<32, true>(A, lda, a_gs, a_rows, W, ldw, w_gs, C, ldc, c_gs, group_off, n_groups, M, N, K, gate, ld_gate, gate_gs, gate_ns, row_scale, scale_by_place, stream)
+                       : launch_mma<64, true>(A, lda, a_gs, a_rows, W, ldw, w_gs, C, ldc, c_gs, group_off, n_groups, M, N, K, gate, ld_gate, gate_gs, gate_ns, row_scale, scale_by_place, stream);
+        return few ? launch_mma<32, false>(A, lda, a_gs, a_rows, W, ldw, w_gs, C, ldc, c_gs, group_off, n_groups, M, N, K, gate, ld_gate, gate_gs, gate_ns, row_scale, scale_by_place, stream)
+                   : launch_mma<64, false>(A, lda, a_gs, a_rows, W, ldw, w_gs, C, ldc, c_gs, group_off, n_groups, M, N, K, gate, ld_gate, gate_gs, gate_ns, row_scale, scale_by_place, stream);
     }
-    if (row_scale) return IL_UNSUPPORTED;         // a factor per row: the tensor-core kernel's epilogue only
     dim3 grid((N + 63) / 64, group_off ? il_gemm_grouped_max_tiles(M, n_groups) : (M + 63) / 64, group_off ? 1 : n_groups);
     if (grid.y > 65535 || grid.z > 65535) return IL_UNSUPPORTED;
 #define GG_LAUNCH(TA, G)                                                                                                                 \
     IL_LAUNCH((gemm_grouped_kernel<TA, G>), grid, 256, 0, stream, (const TA*)A, lda, a_gs, a_rows, (const TA*)W, ldw, w_gs, (TA*)C, ldc, \
-              c_gs, group_off, n_groups, M, N, K, (const TA*)gate, ld_gate, gate_gs)
+              c_gs, group_off, n_groups, M, N, K, (const TA*)gate, ld_gate, gate_gs, gate_ns, row_scale, scale_by_place)
     if (act_kind == IL_F32) {
         if (glu) GG_LAUNCH(float, true); else GG_LAUNCH(float, false);
     } else if (act_kind == IL_BF16) {

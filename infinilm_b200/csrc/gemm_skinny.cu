@@ -64,13 +64,13 @@ __device__ __forceinline__ void gs_norm_finish(float* rstd_s, const float (&pv)[
     }
 }
 
-// NT: 8-row groups of x (1: M <= 8, 2: M <= 16). GLU: 0 plain, 1 SwiGLU, 2 the same with the tanh form of GELU as the gate (W holds N gate rows, then N up rows). U: blocks in flight.
+// NT: 8-row groups of x (1: M <= 8, 2: M <= 16). GLU: 0 plain, 1 SwiGLU, 2 the same with the tanh form of GELU as the gate, 3 with the clamped gate (act_limit, act_alpha) (W holds N gate rows, then N up rows). U: blocks in flight.
 // NRM: the activations may come without their norm's 1/rms (`ni`); the SwiGLU form always can, the plain form as a variant of its own.
 template <int NT, int GLU, int U, typename TO, bool NRM = (GLU != 0)>
 __global__ void __launch_bounds__(GS_WARPS * 32, 2) gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, int ldx,
                                                                     const __nv_bfloat16* __restrict__ W, int ldw, TO* __restrict__ out,
                                                                     int ldo, const float* __restrict__ bias, float alpha, int M, int N, int K,
-                                                                    const GsNormIn ni) {
+                                                                    const GsNormIn ni, float act_limit, float act_alpha) {
     constexpr int NW = 1;
     constexpr int ROWS = GLU ? 8 : 16;            // outputs per activation row and tile: 16 rows, or 8 gate rows with their 8 up rows
     __shared__ float part[GS_WARPS][NW][NT][16][8];
@@ -155,7 +155,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32, 2) gemm_skinny_kernel(const __n
         float y = __fmaf_rn(an, s0, bias ? bias[n] : 0.f);      // spelled out as one fused multiply-add: the same bits from every build of this line
         if (GLU) {
             const float u = __fmaf_rn(an, s1, bias ? bias[N + n] : 0.f);
-            y = GLU == 2 ? il_gelu_tanh_mul_fast(y, u) : il_silu_mul_fast(y, u);
+            y = GLU == 3 ? il_clamped_glu_fast(y, u, act_limit, act_alpha) : GLU == 2 ? il_gelu_tanh_mul_fast(y, u) : il_silu_mul_fast(y, u);
         }
         gs_store<TO>(out + (size_t)m * ldo + n, y);
     }
@@ -163,20 +163,21 @@ __global__ void __launch_bounds__(GS_WARPS * 32, 2) gemm_skinny_kernel(const __n
 
 template <int NT, int GLU, typename TO, bool NRM = (GLU != 0)>
 static cudaError_t gs_launch(const void* x, int ldx, const void* W, int ldw, void* out, int ldo, const float* bias, float alpha, int M, int N,
-                      int K, cudaStream_t stream, const GsNormIn& ni = GsNormIn{nullptr, 0, 0.f, 0.f}) {
+                      int K, cudaStream_t stream, const GsNormIn& ni = GsNormIn{nullptr, 0, 0.f, 0.f}, float act_limit = 0.f,
+                      float act_alpha = 0.f) {
     constexpr int U = NT == 1 ? 8 : 4;
     constexpr int ROWS = GLU ? 8 : 16;
     return il_launch(gemm_skinny_kernel<NT, GLU, U, TO, NRM>, dim3((N + ROWS - 1) / ROWS), dim3(GS_WARPS * 32), 0, stream,
-              (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)out, ldo, bias, alpha, M, N, K, ni);
+              (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)out, ldo, bias, alpha, M, N, K, ni, act_limit, act_alpha);
 }
 
 // glu = 1: W is [2N, K] (N gate rows, then N up rows), bias [2N], out[M,N] = silu(alpha*x.Wg^T + bg) * (alpha*x.Wu^T + bu);
-// glu = 2: the same with gelu_tanh in place of silu.
+// glu = 2: the same with gelu_tanh in place of silu; glu = 3: the clamped gate with its two numbers.
 // norm_partial (may be null): x is residual * norm weight and still wants its 1/rms, from these sums of squares
 // [M][n_partial] (n_partial <= 256, H = the width they were summed over).
 IL_EXPORT int il_gemm_skinny(const void* x, int ldx, const void* W, int ldw, void* out, int out_kind, int ldo, const float* bias,
                              float alpha, int M, int N, int K, int glu, const float* norm_partial, int n_partial, int norm_h,
-                             float norm_eps, cudaStream_t stream) {
+                             float norm_eps, float act_limit, float act_alpha, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return IL_OK;
     if (norm_partial && (n_partial <= 0 || n_partial > GS_NORM_MAX_PARTIALS || norm_h <= 0)) return IL_UNSUPPORTED;
     const GsNormIn ni{norm_partial, n_partial, norm_partial ? 1.f / (float)norm_h : 0.f, norm_eps};
@@ -185,14 +186,16 @@ IL_EXPORT int il_gemm_skinny(const void* x, int ldx, const void* W, int ldw, voi
     if (glu && out_kind != IL_BF16) return IL_UNSUPPORTED;
     cudaError_t e;
     if (M <= 8) {
-        if (glu == 2) e = gs_launch<1, 2, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
+        if (glu == 3) e = gs_launch<1, 3, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni, act_limit, act_alpha);
+        else if (glu == 2) e = gs_launch<1, 2, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (glu) e = gs_launch<1, 1, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (norm_partial && out_kind == IL_BF16) e = gs_launch<1, 0, __nv_bfloat16, true>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (norm_partial) e = gs_launch<1, 0, float, true>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (out_kind == IL_BF16) e = gs_launch<1, 0, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream);
         else e = gs_launch<1, 0, float>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream);
     } else {
-        if (glu == 2) e = gs_launch<2, 2, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
+        if (glu == 3) e = gs_launch<2, 3, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni, act_limit, act_alpha);
+        else if (glu == 2) e = gs_launch<2, 2, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (glu) e = gs_launch<2, 1, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (norm_partial && out_kind == IL_BF16) e = gs_launch<2, 0, __nv_bfloat16, true>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (norm_partial) e = gs_launch<2, 0, float, true>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);

@@ -71,6 +71,94 @@ IL_EXPORT int il_latent_norm_store(const void* proj, int act_kind, int row_strid
     return IL_OK;
 }
 
+// ---- a latent with a rotated key part beside it ---------------------------------------------------------------------------
+// Per token: the latent (n_b columns at off_b) is divided by its root mean square and multiplied by w_b; the `rd` columns
+// behind it are one key part for all heads, of which the first `rot` dimensions turn by pos * freq[i] (cosine and sine times
+// mscale; pairs (2i, 2i + 1) or (i, i + rot / 2)) and the others pass. Latent, turned part and zeros up to hd columns go to the
+// token's slot of the cache, K plane and V plane alike. Every head's query has its rotated part behind its other
+// `qd` columns (head j at off_q + j * (qd + rd)): turned likewise, it goes to q_out[t, j * hd + n_b ..], zeros behind it; the
+// columns in front of it are the business of the product that brings the query's other part to the latent's width.
+// Angles are made in double precision and reduced to one turn before sine and cosine are taken in f32: an f32 product of
+// position and frequency would be off by a rounding of the whole angle. Norm and rotation f32. One block per token.
+#define LR_MAX_ROT 1024
+template <typename TA>
+__global__ void latent_rope_store_kernel(const TA* proj, int row_stride, int off_q, int nh, int qd, int off_b, int n_b, int rd, int hd,
+                                         const void* __restrict__ w_b, int w_kind, float eps, int rot, const double* __restrict__ freq, float mscale,
+                                         int interleaved, TA* __restrict__ q_out, const int* __restrict__ tok_pos, const int* __restrict__ tok_entry,
+                                         const int* __restrict__ block_table, int bt_stride, TA* __restrict__ cache, int page_size) {
+    __shared__ float red[32];
+    __shared__ float s_cos[LR_MAX_ROT / 2], s_sin[LR_MAX_ROT / 2];
+    const int t = blockIdx.x;
+    const int pos = tok_pos[t];
+    TA* kdst = nullptr;
+    const size_t plane = (size_t)page_size * hd;
+    if (cache) {
+        const int page = block_table[(size_t)tok_entry[t] * bt_stride + pos / page_size];
+        if (page >= 0) kdst = cache + (size_t)page * 2 * plane + (size_t)(pos % page_size) * hd;      // (the host reserves every page a step touches)
+    }
+    const int half = rot >> 1;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const double turn = 6.283185307179586476925;
+        double a = (double)pos * freq[i];
+        a -= turn * rint(a / turn);
+        float s, c;
+        sincosf((float)a, &s, &c);
+        s_sin[i] = s * mscale, s_cos[i] = c * mscale;
+    }
+    il_pdl_begin();
+    const TA* row = proj + (size_t)t * row_stride;
+    float sb = 0.f;
+    for (int i = threadIdx.x; i < n_b; i += blockDim.x) {
+        const float x = il_to_f(row[off_b + i]);
+        sb += x * x;
+    }
+    sb = il_block_sum(sb, red);                   // (its barriers also stand between the writing and the reading of the angles)
+    const float rb = 1.f / sqrtf(sb / (float)n_b + eps);
+    auto turned = [&](const TA* x, int d) -> float {
+        if (d >= rot) return il_to_f(x[d]);
+        const bool low = interleaved ? !(d & 1) : d < half;
+        const int i = interleaved ? d >> 1 : (low ? d : d - half), mate = interleaved ? d ^ 1 : (low ? d + half : d - half);
+        const float a = il_to_f(x[d]), b = il_to_f(x[mate]), s = s_sin[i], c = s_cos[i];
+        return low ? a * c - b * s : a * c + b * s;
+    };
+    if (kdst) {
+        for (int i = threadIdx.x; i < hd; i += blockDim.x) {
+            const float f = i < n_b ? il_to_f(row[off_b + i]) * rb * il_load_any(w_b, w_kind, i) : i < n_b + rd ? turned(row + off_b + n_b, i - n_b) : 0.f;
+            const TA v = il_from_f<TA>(f);
+            kdst[i] = v;
+            kdst[plane + i] = v;
+        }
+    }
+    const int tail = hd - n_b;
+    for (int idx = threadIdx.x; idx < nh * tail; idx += blockDim.x) {
+        const int j = idx / tail, d = idx - j * tail;
+        q_out[((size_t)t * nh + j) * hd + n_b + d] = il_from_f<TA>(d < rd ? turned(row + off_q + (size_t)j * (qd + rd) + qd, d) : 0.f);
+    }
+}
+
+IL_EXPORT int il_latent_rope_store(const void* proj, int act_kind, int row_stride, int off_q, int nh, int qd, int off_b, int n_b, int rd, int hd,
+                                   const void* w_b, int w_kind, float eps, int rot, const double* freq, float mscale, int interleaved, void* q_out,
+                                   const int* tok_pos, const int* tok_entry, const int* block_table, int bt_stride, void* cache, int page_size, int T,
+                                   cudaStream_t stream) {
+    if (T <= 0) return IL_OK;
+    if (nh <= 0 || qd < 0 || n_b <= 0 || rd < 0 || hd < n_b + rd || page_size <= 0 || !w_b || !q_out) return IL_BAD_ARG;
+    if (rot < 0 || (rot & 1) || rot > rd || (rot > 0 && !freq)) return IL_BAD_ARG;
+    if (rot > LR_MAX_ROT) return IL_UNSUPPORTED;
+    const int work = hd + nh * (hd - n_b);
+    const int threads = work >= 1024 ? 256 : 128;
+    if (act_kind == IL_F32)
+        IL_LAUNCH(latent_rope_store_kernel<float>, T, threads, 0, stream, (const float*)proj, row_stride, off_q, nh, qd, off_b, n_b, rd, hd, w_b, w_kind,
+                  eps, rot, freq, mscale, interleaved, (float*)q_out, tok_pos, tok_entry, block_table, bt_stride, (float*)cache, page_size);
+    else if (act_kind == IL_BF16)
+        IL_LAUNCH(latent_rope_store_kernel<__nv_bfloat16>, T, threads, 0, stream, (const __nv_bfloat16*)proj, row_stride, off_q, nh, qd, off_b, n_b, rd,
+                  hd, w_b, w_kind, eps, rot, freq, mscale, interleaved, (__nv_bfloat16*)q_out, tok_pos, tok_entry, block_table, bt_stride,
+                  (__nv_bfloat16*)cache, page_size);
+    else
+        return IL_BAD_ARG;
+    IL_LAUNCH_CHECK();
+    return IL_OK;
+}
+
 // y[t, c] *= sigmoid(g[t, c]) for rows of `n` columns (y contiguous, g with a row stride): the heads' gate where the product
 // before it was the library's and has no epilogue of ours.
 template <typename TA>

@@ -26,14 +26,44 @@ __device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
 }
 
 // One warp picks the `top` largest of a token's E logits in shared memory (overwritten), the lower expert winning a
-// tie, and writes the experts and their weights. Two rules:
+// tie, and writes the experts and their weights. Three rules:
 //   rule 0: the largest logits are chosen; the weights are the softmax over the chosen logits alone.
+//   rule 2: scores s = sigmoid of the logits, each on its own; the largest s + corr are chosen (without `corr`: the largest logits,
+//           the same order where no two scores round to one number); the weights are the chosen experts' s, times out_scale.
 //   rule 1: scores s = softmax of the logits over all E; the largest s + corr are chosen (`corr`: one number per expert, or
 //           null); the weights are the chosen experts' s over their sum (+ 1e-20), times out_scale.
 __device__ __forceinline__ void moe_pick(float* z, int E, int top, int* __restrict__ idx, float* __restrict__ wt, int lane, int rule = 0,
                                          const void* __restrict__ corr = nullptr, int c_kind = 0, float out_scale = 1.f) {
     float chosen_v[MOE_MAX_TOP];
     float vmax = 0.f, den = 0.f;
+    if (rule == 2) {
+        for (int k = 0; k < top; ++k) {
+            float bv = -INFINITY;
+            int bi = 0x7fffffff;
+            for (int e = lane; e < E; e += 32) {
+                const float ze = z[e];
+                if (ze == -INFINITY) continue;    // chosen already
+                const float v = corr ? 1.f / (1.f + expf(-ze)) + il_load_any(corr, c_kind, e) : ze;
+                if (v > bv || (v == bv && e < bi)) bv = v, bi = e;
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+                const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+                if (ov > bv || (ov == bv && oi < bi)) bv = ov, bi = oi;
+            }
+            if (bi >= E) bi = 0;                  // every score NaN: still a valid expert
+            const float sb = 1.f / (1.f + expf(-z[bi]));
+            __syncwarp();
+            if (lane == 0) {
+                idx[k] = bi;
+                wt[k] = sb * out_scale;
+                z[bi] = -INFINITY;
+            }
+            __syncwarp();
+        }
+        return;
+    }
     if (rule == 1) {
         float mx = -INFINITY;
         for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
@@ -208,16 +238,17 @@ __global__ void __launch_bounds__(WARPS * 32) moe_select_kernel(const float* __r
     il_pdl_begin();
     if (t >= T) return;
     float* zs = sm + (size_t)warp * E;
-    // (rule 1: the bias is no part of the logits; it joins the scores where the experts are chosen)
+    // (rules 1 and 2: the bias is no part of the logits; it joins the scores where the experts are chosen)
     for (int e = lane; e < E; e += 32) zs[e] = z[(size_t)t * ldz + e] + ((bias && rule == 0) ? il_load_any(bias, b_kind, e) : 0.f);
     __syncwarp();
     moe_pick(zs, E, top, idx + (size_t)t * top, wt + (size_t)t * top, lane, rule, bias, b_kind, out_scale);
 }
 
 // The body of the sort, by one whole block; `sh`: 2 * E ints of shared memory. (idx is not declared __restrict__: the
-// fused kernel below reads what its own warps have just written.)
+// fused kernel below reads what its own warps have just written.) `wt_of_pos` (or null) receives every place's weight: where a
+// choice's weight belongs to the expert's input, the products take it as a factor per place.
 __device__ __forceinline__ void moe_sort_body(int* sh, const int* idx, int n_slots, int top, int E, int* __restrict__ group_off,
-                                              int* __restrict__ pos_of_slot, int* __restrict__ row_of_pos) {
+                                              int* __restrict__ pos_of_slot, int* __restrict__ row_of_pos, const float* wt, float* __restrict__ wt_of_pos) {
     int* cnt = sh;
     int* cur = sh + E;
     for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
@@ -244,15 +275,17 @@ __device__ __forceinline__ void moe_sort_body(int* sh, const int* idx, int n_slo
             const int p = atomicAdd(&cur[e], 1);
             pos_of_slot[i] = p;
             row_of_pos[p] = i / top;
+            if (wt_of_pos) wt_of_pos[p] = wt[i];
         }
     }
 }
 
 __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* idx, int n_slots, int top, int E, int* __restrict__ group_off,
-                                                        int* __restrict__ pos_of_slot, int* __restrict__ row_of_pos) {
+                                                        int* __restrict__ pos_of_slot, int* __restrict__ row_of_pos, const float* wt,
+                                                        float* __restrict__ wt_of_pos) {
     extern __shared__ int sh[];                   // [E] counts, then [E] cursors
     il_pdl_begin();
-    moe_sort_body(sh, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos);
+    moe_sort_body(sh, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
 }
 
 // ---- the router of a decode step (a few bfloat16 rows) as two short kernels --------------------------------------------
@@ -311,9 +344,10 @@ __global__ void __launch_bounds__(ML_WARPS * 32) moe_logits_kernel(const __nv_bf
 }
 
 // Chooses for every token (a warp a token, in turns) from logits z [T, E], then sorts the slots: one block.
-__global__ void __launch_bounds__(1024) moe_select_sort_kernel(const float* z, int ldz, int* idx, float* __restrict__ wt, int T, int E, int top,
+__global__ void __launch_bounds__(1024) moe_select_sort_kernel(const float* z, int ldz, int* idx, float* wt, int T, int E, int top,
                                                                int* __restrict__ group_off, int* __restrict__ pos_of_slot, int* __restrict__ row_of_pos,
-                                                               int rule, const void* __restrict__ corr, int c_kind, float out_scale) {
+                                                               int rule, const void* __restrict__ corr, int c_kind, float out_scale,
+                                                               float* __restrict__ wt_of_pos) {
     extern __shared__ __align__(16) float sm[];   // [32][E] logits of the warps' tokens, then 2 * E ints for the sort
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     il_pdl_begin();
@@ -325,7 +359,7 @@ __global__ void __launch_bounds__(1024) moe_select_sort_kernel(const float* z, i
         __syncwarp();
     }
     __syncthreads();                              // the choices, written to memory by this block's warps, are read below
-    moe_sort_body(reinterpret_cast<int*>(sm + (size_t)32 * E), idx, T * top, top, E, group_off, pos_of_slot, row_of_pos);
+    moe_sort_body(reinterpret_cast<int*>(sm + (size_t)32 * E), idx, T * top, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
 }
 
 __device__ __forceinline__ float4 ld4c(const float* p) { return *reinterpret_cast<const float4*>(p); }
@@ -358,7 +392,7 @@ __global__ void moe_combine_kernel(const TA* y, const int* pos_of_slot, const fl
     if (threadIdx.x < top) {                      // the token's places and weights once, not once per column
         const int p = pos_of_slot[(size_t)t * top + threadIdx.x];
         sp[threadIdx.x] = (group_off && p >= group_off[n_real]) ? -1 : p;       // -1: the input row itself
-        sw[threadIdx.x] = wt[(size_t)t * top + threadIdx.x];
+        sw[threadIdx.x] = wt ? wt[(size_t)t * top + threadIdx.x] : 1.f;      // (null: the weights went into the experts' inputs)
     }
     __syncthreads();
     const float sg = (shared_rows && sgate) ? 1.f / (1.f + expf(-sgate[(size_t)t * ld_sg])) : 1.f;
@@ -509,11 +543,12 @@ IL_EXPORT int il_moe_route(const void* x, int act_kind, int ldx, const void* w, 
 }
 
 // rule 0: the `top` largest of z + bias, weights their softmax. rule 1: scores softmax(z) over all E, the largest score + bias
-// chosen, weights the chosen scores over their sum, times out_scale (see moe_pick).
+// chosen, weights the chosen scores over their sum, times out_scale. rule 2: scores sigmoid(z), weights the chosen scores, times
+// out_scale (see moe_pick).
 IL_EXPORT int il_moe_select(const float* z, int ldz, const void* bias, int b_kind, int* idx, float* wt, int T, int E, int top, int rule,
                             float out_scale, cudaStream_t stream) {
     if (T <= 0) return IL_OK;
-    if (E <= 0 || top <= 0 || top > E || top > MOE_MAX_TOP || ldz < E || (rule != 0 && rule != 1)) return IL_BAD_ARG;
+    if (E <= 0 || top <= 0 || top > E || top > MOE_MAX_TOP || ldz < E || rule < 0 || rule > 2) return IL_BAD_ARG;
     constexpr int WARPS = 8;
     const size_t smem = (size_t)WARPS * E * sizeof(float);
     if (smem > 200 * 1024) return IL_UNSUPPORTED;
@@ -532,9 +567,9 @@ IL_EXPORT int il_moe_select(const float* z, int ldz, const void* bias, int b_kin
 // choice (a gate that is a function of the same rows). rule, out_scale: see il_moe_select.
 IL_EXPORT int il_moe_route_sort_small(const void* x, int ldx, const void* w, const void* bias, int b_kind, float* z, int* idx, float* wt, int T, int H,
                                       int E, int top, const float* sumsq, int n_partial, float eps, float* rstd_out, int* group_off,
-                                      int* pos_of_slot, int* row_of_pos, int extra, int rule, float out_scale, cudaStream_t stream) {
+                                      int* pos_of_slot, int* row_of_pos, int extra, int rule, float out_scale, float* wt_of_pos, cudaStream_t stream) {
     if (T <= 0) return IL_OK;
-    if (H <= 0 || E <= 0 || top <= 0 || top > E || top > MOE_MAX_TOP || (sumsq && n_partial <= 0) || extra < 0 || (rule != 0 && rule != 1) ||
+    if (H <= 0 || E <= 0 || top <= 0 || top > E || top > MOE_MAX_TOP || (sumsq && n_partial <= 0) || extra < 0 || rule < 0 || rule > 2 ||
         (extra > 0 && bias && rule == 0))
         return IL_BAD_ARG;
     const size_t smem = (size_t)32 * E * sizeof(float) + (size_t)2 * E * sizeof(int);
@@ -547,16 +582,18 @@ IL_EXPORT int il_moe_route_sort_small(const void* x, int ldx, const void* w, con
     IL_LAUNCH(moe_logits_kernel, dim3((EZ + ML_WARPS - 1) / ML_WARPS, T), ML_WARPS * 32, 0, stream, (const __nv_bfloat16*)x, ldx,
               (const __nv_bfloat16*)w, rule == 0 ? bias : (const void*)nullptr, b_kind, z, T, H, EZ, sumsq, n_partial, 1.f / (float)H, eps, rstd_out);
     IL_LAUNCH(moe_select_sort_kernel, 1, 1024, smem, stream, (const float*)z, EZ, idx, wt, T, E, top, group_off, pos_of_slot, row_of_pos, rule,
-              rule == 1 ? bias : (const void*)nullptr, b_kind, out_scale);
+              rule != 0 ? bias : (const void*)nullptr, b_kind, out_scale, wt_of_pos);
     IL_LAUNCH_CHECK();
     return IL_OK;
 }
 
-IL_EXPORT int il_moe_sort(const int* idx, int n_slots, int top, int E, int* group_off, int* pos_of_slot, int* row_of_pos, cudaStream_t stream) {
-    if (E <= 0 || top <= 0 || n_slots < 0) return IL_BAD_ARG;
+// wt (n_slots weights in the order of the slots) and wt_of_pos (out, in the order of the places): both or neither.
+IL_EXPORT int il_moe_sort(const int* idx, int n_slots, int top, int E, int* group_off, int* pos_of_slot, int* row_of_pos, const float* wt,
+                          float* wt_of_pos, cudaStream_t stream) {
+    if (E <= 0 || top <= 0 || n_slots < 0 || (wt_of_pos && !wt)) return IL_BAD_ARG;
     const size_t smem = (size_t)2 * E * sizeof(int);
     if (smem > 48 * 1024) return IL_UNSUPPORTED;
-    IL_LAUNCH(moe_sort_kernel, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos);
+    IL_LAUNCH(moe_sort_kernel, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
     IL_LAUNCH_CHECK();
     return IL_OK;
 }

@@ -206,6 +206,130 @@ __global__ void __launch_bounds__(256) norm_add_kernel(float* resid, const TA* b
     }
 }
 
+// ---- the norm on the branch, the residual add and the next norm in one pass --------------------------------------------
+//   b         = branch[r], or the sum over a token's routed rows: sum_k wt[r, k] * y[pos[r, k]]  (wt null: plain sum)
+//   resid[r] += b / sqrt(mean(b^2) + eps_b) * w_b                                   (f32)
+//   out[r]    = resid[r] / sqrt(mean(resid[r]^2) + eps_n) * w_n                     (out null: only the add)
+// What lies between two sublayers of a model with a norm before and one after each. One block per row with a fixed thread
+// count; a thread's columns (v = thread, thread + 256, ... groups of VW) stay in registers between the passes.
+template <typename TA, int VW> struct NanVec;
+template <typename TA> struct NanVec<TA, 4> {
+    static __device__ __forceinline__ float4 ld(const TA* p) { return ld4(p); }
+    static __device__ __forceinline__ void st(TA* p, float4 v) { st4(p, v); }
+};
+template <typename TA> struct NanVec<TA, 1> {
+    static __device__ __forceinline__ float4 ld(const TA* p) { return make_float4(il_to_f(*p), 0.f, 0.f, 0.f); }
+    static __device__ __forceinline__ void st(TA* p, float4 v) { *p = il_from_f<TA>(v.x); }
+};
+template <int VW> __device__ __forceinline__ float4 nan_w(const void* w, int kind, int h) {
+    if (VW == 4) return kind == IL_F32 ? ld4((const float*)w + h) : ld4((const __nv_bfloat16*)w + h);
+    return make_float4(il_load_any(w, kind, h), 0.f, 0.f, 0.f);
+}
+#define NAN_MAX_TOP 32
+template <typename TA, int VW, int MAXV>
+__global__ void __launch_bounds__(256) norm_add_norm_kernel(float* resid, const TA* branch, const int* pos, const float* wt, int top,
+                                                            const void* __restrict__ wb, int wb_kind, float eps_b, const void* __restrict__ wn,
+                                                            int wn_kind, float eps_n, TA* __restrict__ out, int H) {
+    __shared__ float red[32];
+    __shared__ int sp[NAN_MAX_TOP];
+    __shared__ float sw[NAN_MAX_TOP];
+    const int r = blockIdx.x, nv = (H + VW - 1) / VW;
+    // the norms' weights do not come from the kernel before this one: read while it still runs
+    float4 a[MAXV], b[MAXV];
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+        const int v = threadIdx.x + k * 256;
+        a[k] = v < nv ? nan_w<VW>(wb, wb_kind, v * VW) : make_float4(0.f, 0.f, 0.f, 0.f);
+        b[k] = (out && v < nv) ? nan_w<VW>(wn, wn_kind, v * VW) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    il_pdl_wait();
+    if (pos) {
+        if (threadIdx.x < top) {
+            sp[threadIdx.x] = pos[(size_t)r * top + threadIdx.x];
+            sw[threadIdx.x] = wt ? wt[(size_t)r * top + threadIdx.x] : 1.f;
+        }
+        __syncthreads();
+    }
+    float* rr = resid + (size_t)r * H;
+    float4 x[MAXV], c[MAXV];
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+        const int v = threadIdx.x + k * 256;
+        x[k] = v < nv ? NanVec<float, VW>::ld(rr + v * VW) : make_float4(0.f, 0.f, 0.f, 0.f);
+        c[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (v < nv && !pos) c[k] = NanVec<TA, VW>::ld(branch + (size_t)r * H + v * VW);
+    }
+    if (pos) {                                    // the rows of a token's choices, in the order of the choices
+        for (int i = 0; i < top; ++i) {
+            const TA* y = branch + (size_t)sp[i] * H;
+            const float w = sw[i];
+#pragma unroll
+            for (int k = 0; k < MAXV; ++k) {
+                const int v = threadIdx.x + k * 256;
+                if (v < nv) {
+                    const float4 t = NanVec<TA, VW>::ld(y + v * VW);
+                    c[k].x = fmaf(w, t.x, c[k].x), c[k].y = fmaf(w, t.y, c[k].y), c[k].z = fmaf(w, t.z, c[k].z), c[k].w = fmaf(w, t.w, c[k].w);
+                }
+            }
+        }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) ss += c[k].x * c[k].x + c[k].y * c[k].y + c[k].z * c[k].z + c[k].w * c[k].w;
+    ss = il_block_sum(ss, red);
+    const float kb = 1.f / sqrtf(ss / (float)H + eps_b);
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+        const int v = threadIdx.x + k * 256;
+        x[k].x = fmaf(kb * c[k].x, a[k].x, x[k].x), x[k].y = fmaf(kb * c[k].y, a[k].y, x[k].y);
+        x[k].z = fmaf(kb * c[k].z, a[k].z, x[k].z), x[k].w = fmaf(kb * c[k].w, a[k].w, x[k].w);
+        if (v < nv) NanVec<float, VW>::st(rr + v * VW, x[k]);
+        ss += x[k].x * x[k].x + x[k].y * x[k].y + x[k].z * x[k].z + x[k].w * x[k].w;
+    }
+    if (!out) return;
+    ss = il_block_sum(ss, red);
+    const float kn = 1.f / sqrtf(ss / (float)H + eps_n);
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+        const int v = threadIdx.x + k * 256;
+        if (v < nv)
+            NanVec<TA, VW>::st(out + (size_t)r * H + v * VW, make_float4(x[k].x * kn * b[k].x, x[k].y * kn * b[k].y, x[k].z * kn * b[k].z, x[k].w * kn * b[k].w));
+    }
+}
+
+template <typename TA>
+static int nan_launch(float* resid, const void* branch, const int* pos, const float* wt, int top, const void* wb, int wb_kind, float eps_b,
+                      const void* wn, int wn_kind, float eps_n, void* out, int n_rows, int H, cudaStream_t stream) {
+    const bool vec = (H & 3) == 0 && (((uintptr_t)resid | (uintptr_t)branch | (uintptr_t)wb | (uintptr_t)wn | (uintptr_t)out) & 15) == 0;
+#define NAN_GO(VW, MAXV)                                                                                                                     \
+    IL_LAUNCH((norm_add_norm_kernel<TA, VW, MAXV>), n_rows, 256, 0, stream, resid, (const TA*)branch, pos, wt, top, wb, wb_kind, eps_b, wn, \
+              wn_kind, eps_n, (TA*)out, H)
+    if (vec && H <= 256 * 4) NAN_GO(4, 1);
+    else if (vec && H <= 256 * 4 * 2) NAN_GO(4, 2);
+    else if (vec && H <= 256 * 4 * 4) NAN_GO(4, 4);
+    else if (vec && H <= 256 * 4 * 8) NAN_GO(4, 8);
+    else if (H <= 256 * 4) NAN_GO(1, 4);
+    else if (H <= 256 * 16) NAN_GO(1, 16);
+    else return IL_UNSUPPORTED;
+#undef NAN_GO
+    return IL_OK;
+}
+
+// branch: [n_rows, H], or - with `pos` [n_rows, top] - the rows y that the places in `pos` name.
+IL_EXPORT int il_norm_add_norm(float* resid, const void* branch, const int* pos, const float* wt, int top, const void* wb, int wb_kind, float eps_b,
+                               const void* wn, int wn_kind, float eps_n, void* out, int act_kind, int n_rows, int H, cudaStream_t stream) {
+    if (n_rows <= 0) return IL_OK;
+    if (H <= 0 || !branch || !wb || (out && !wn) || (pos && (top <= 0 || top > NAN_MAX_TOP))) return IL_BAD_ARG;
+    int rc;
+    if (act_kind == IL_F32) rc = nan_launch<float>(resid, branch, pos, wt, top, wb, wb_kind, eps_b, wn, wn_kind, eps_n, out, n_rows, H, stream);
+    else if (act_kind == IL_BF16) rc = nan_launch<__nv_bfloat16>(resid, branch, pos, wt, top, wb, wb_kind, eps_b, wn, wn_kind, eps_n, out, n_rows, H, stream);
+    else return IL_BAD_ARG;
+    if (rc != IL_OK) return rc;
+    IL_LAUNCH_CHECK();
+    return IL_OK;
+}
+
 // rows of f32 copied into the activations' type (the first sublayer's input, where no norm_add ran before it)
 template <typename TA>
 __global__ void cast_rows_kernel(const float* x, TA* out, size_t total) {

@@ -153,18 +153,32 @@ def add_rmsnorm(resid: torch.Tensor, branch: Optional[torch.Tensor], branch_scal
              kind_of(out.dtype), _ptr(rows), n, H, _ptr(vec), H if vec is not None and vec.dim() == 2 else 0, _stream()), "add_rmsnorm")
 
 
-ACT_SILU, ACT_GELU_TANH = 1, 2                    # the gate of a gated feed-forward
+ACT_SILU, ACT_GELU_TANH, ACT_CLAMPED = 1, 2, 3    # the gate of a gated feed-forward
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, act: int = ACT_SILU) -> None:
-    """out[t,i] = act(gate_up[t,i]) * gate_up[t,I+i]; act: SiLU or the tanh form of GELU."""
-    _need_cuda(gate_up, out)
+def _act_args(act: int, act_params):
+    """The clamped gate's two numbers (limit, alpha); the other gates have none."""
+    if int(act) != ACT_CLAMPED:
+        return 0.0, 0.0
+    if act_params is None or not float(act_params[0]) > 0.0:
+        raise KernelError("the clamped gate needs act_params (limit > 0, alpha)")
+    return float(act_params[0]), float(act_params[1])
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, act: int = ACT_SILU, act_params=None, row_scale: Optional[torch.Tensor] = None) -> None:
+    """out[t,i] = act(gate_up[t,i]) * gate_up[t,I+i]; act: SiLU, the tanh form of GELU, or ACT_CLAMPED with act_params
+    (limit, alpha): g sigmoid(alpha g) (u + 1) with g = min(gate, limit) and u kept within -limit .. limit.
+    row_scale: float32 [T], multiplied into a row's gate and up products before anything else."""
+    _need_cuda(gate_up, out, row_scale)
+    if row_scale is not None and (row_scale.dtype != torch.float32 or row_scale.numel() < gate_up.shape[0] or not row_scale.is_contiguous()):
+        raise KernelError("swiglu: row_scale float32 [T]")
     T, I2 = gate_up.shape
     if I2 % 2 or out.shape != (T, I2 // 2) or out.dtype != gate_up.dtype:
         raise KernelError("swiglu: gate_up [T,2I], out [T,I] of the same dtype")
     _contig("gate_up", gate_up), _contig("out", out)
-    f = _fn("swiglu", "il_swiglu", [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p])
-    _check(f(_ptr(gate_up), _ptr(out), kind_of(out.dtype), T, I2 // 2, act, _stream()), "swiglu")
+    f = _fn("swiglu", "il_swiglu", [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p, _c_void_p])
+    limit, alpha = _act_args(act, act_params)
+    _check(f(_ptr(gate_up), _ptr(out), kind_of(out.dtype), T, I2 // 2, int(act), limit, alpha, _ptr(row_scale), _stream()), "swiglu")
 
 
 def add_bias(y: torch.Tensor, bias: torch.Tensor) -> None:
@@ -203,13 +217,14 @@ def rope_store(qkv: torch.Tensor, tok_pos: torch.Tensor, tok_entry: torch.Tensor
 def attention_plain(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                     tok_pos: torch.Tensor, tok_entry: torch.Tensor, page_size: int, n_heads: int,
                     n_kv_heads: int, head_dim: int, scale: float, window: Optional[int] = None,
-                    sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None) -> None:
+                    sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None, sigmoid: bool = False) -> None:
     """Causal attention of every token of `qkv` over its request's cache pages (plain kernel). `qkv` needs the query
     heads only (keys and values are read from the cache). `sink`: float32 [heads], a score per head that joins the
     softmax's denominator without a value. `dist_bias`: float32 [far + 1, heads], added to the scaled score of a key n
-    positions back as dist_bias[min(n, far), head]."""
+    positions back as dist_bias[min(n, far), head]. `sigmoid`: a key's weight is the sigmoid of its score, not normalised over
+    the keys (no softmax, so no sink)."""
     _need_cuda(qkv, out, cache, block_table, tok_pos, tok_entry, sink, dist_bias)
-    _check_sink(sink, n_heads)
+    _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)
     T = qkv.shape[0]
     if out.shape != (T, n_heads * head_dim) or out.dtype != qkv.dtype or cache.dtype != qkv.dtype:
@@ -219,14 +234,16 @@ def attention_plain(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, b
     _contig("qkv", qkv), _contig("out", out), _contig("cache", cache), _contig("block_table", block_table)
     f = _fn("attn_plain", "il_attn_plain", [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
                                             _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
-                                            _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p])
+                                            _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p])
     _check(f(_ptr(qkv), kind_of(qkv.dtype), qkv.shape[1], _ptr(out), _ptr(cache), _ptr(block_table),
              block_table.shape[1], _ptr(tok_pos), _ptr(tok_entry), page_size, T, n_heads, n_kv_heads, head_dim,
-             scale, int(window or 0), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, _stream()),
+             scale, int(window or 0), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), _stream()),
            "attention_plain")
 
 
-def _check_sink(sink: Optional[torch.Tensor], n_heads: int) -> None:
+def _check_sink(sink: Optional[torch.Tensor], n_heads: int, sigmoid: bool = False) -> None:
+    if sigmoid and sink is not None:
+        raise KernelError("attention: a sink belongs to a softmax's denominator; sigmoid weights have none")
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != n_heads or not sink.is_contiguous()):
         raise KernelError("attention: sink must be a contiguous float32 tensor, one number per query head")
 
@@ -253,6 +270,44 @@ def norm_add(resid: torch.Tensor, branch: torch.Tensor, weight: torch.Tensor, ep
                                        _c_void_p])
     _check(f(_ptr(resid), _ptr(branch), scale, _ptr(weight), kind_of(weight.dtype), eps, _ptr(copy), kind_of(branch.dtype), T, H,
              _stream()), "norm_add")
+
+
+class RoutedRows:
+    """A routed feed-forward's result before its rows are summed: token t's branch is sum_k wt[t, k] * y[pos[t * top + k]]
+    (wt None: a plain sum). Whoever reads the branch next sums the rows itself."""
+    __slots__ = ("y", "pos", "wt", "top")
+
+    def __init__(self, y: torch.Tensor, pos: torch.Tensor, wt: Optional[torch.Tensor], top: int):
+        self.y, self.pos, self.wt, self.top = y, pos, wt, int(top)
+
+
+def norm_add_norm(resid: torch.Tensor, branch, branch_weight: torch.Tensor, branch_eps: float, next_weight: Optional[torch.Tensor] = None,
+                  next_eps: float = 0.0, out: Optional[torch.Tensor] = None) -> None:
+    """resid += branch / sqrt(mean(branch^2) + branch_eps) * branch_weight (float32 [T,H], in place), then, with `out`,
+    out = resid / sqrt(mean(resid^2) + next_eps) * next_weight: what lies between two sublayers of a model with a norm before
+    and one behind each. `branch`: rows [T,H], or `RoutedRows`."""
+    routed = branch if isinstance(branch, RoutedRows) else None
+    y, pos, wt = (routed.y, routed.pos, routed.wt) if routed is not None else (branch, None, None)
+    _need_cuda(resid, y, pos, wt, branch_weight, next_weight, out)
+    T, H = resid.shape
+    if resid.dtype != torch.float32 or branch_weight.numel() != H or y.dim() != 2 or y.shape[1] != H:
+        raise KernelError("norm_add_norm: resid float32 [T,H], branch [T,H], branch_weight [H]")
+    if routed is None and y.shape[0] != T:
+        raise KernelError("norm_add_norm: branch [T,H]")
+    if routed is not None and (pos.dtype != torch.int32 or pos.numel() < T * routed.top or not pos.is_contiguous() or not 0 < routed.top <= MOE_MAX_TOP
+                               or y.shape[0] < T * routed.top
+                               or (wt is not None and (wt.dtype != torch.float32 or tuple(wt.shape) != (T, routed.top) or not wt.is_contiguous()))):
+        raise KernelError("norm_add_norm: routed rows y [T * top, H], pos int32 [T * top], wt float32 [T, top] or None")
+    if out is not None and (next_weight is None or next_weight.numel() != H or tuple(out.shape) != (T, H) or out.dtype != y.dtype or not out.is_contiguous()):
+        raise KernelError("norm_add_norm: out [T,H] of the branch's dtype comes with next_weight [H]")
+    _contig("resid", resid), _contig("branch", y), _contig("branch_weight", branch_weight)
+    if next_weight is not None:
+        _contig("next_weight", next_weight)
+    f = _fn("rmsnorm", "il_norm_add_norm", [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_void_p, _c_int,
+                                            _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_void_p])
+    _check(f(_ptr(resid), _ptr(y), _ptr(pos), _ptr(wt), 0 if routed is None else routed.top, _ptr(branch_weight), kind_of(branch_weight.dtype),
+             branch_eps, _ptr(next_weight if out is not None else None), kind_of(next_weight.dtype) if out is not None else 0, next_eps, _ptr(out),
+             kind_of(y.dtype), T, H, _stream()), "norm_add_norm")
 
 
 HYPER_MAX_STREAMS = 16
@@ -436,16 +491,18 @@ def attention_decode(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
                      entry_kvlen: torch.Tensor, n_decode: int, page_size: int, n_heads: int, n_kv_heads: int,
                      head_dim: int, scale: float, window: Optional[int], pages_per_split: int, n_splits: int,
                      o_part: torch.Tensor, ml_part: torch.Tensor, kv_map: Optional[torch.Tensor] = None,
-                     sink: Optional[torch.Tensor] = None, v_is_k: bool = False, dist_bias: Optional[torch.Tensor] = None) -> None:
+                     sink: Optional[torch.Tensor] = None, v_is_k: bool = False, dist_bias: Optional[torch.Tensor] = None,
+                     sigmoid: bool = False) -> None:
     """bfloat16 split-KV attention of token rows [0, n_decode) (entry i = row i, one token each), then the merge of
     the splits (a second launch; with n_splits = 1 there is none and the attention kernel writes `out` itself). A row whose length is 0 gets zeros; a block-table entry below 0 is never followed.
     pages_per_split 0: each request's pages are divided evenly over the n_splits splits.
     kv_map: the cache's tensor map from `kv_tensor_map` (pages then come in by TMA tensor copies).
     v_is_k: the caller vouches that the V plane of every page repeats its K plane (a latent that is key and value at once);
     with a tensor map only the K plane is then read, half the bytes.
+    sigmoid: a key's weight is the sigmoid of its score, not normalised over the keys.
     Scratch: o_part float32 [n_decode*heads*n_splits*head_dim], ml_part float32 [n_decode*heads*n_splits*2]."""
     _need_cuda(qkv, out, cache, block_table, entry_kvlen, o_part, ml_part, sink, dist_bias)
-    _check_sink(sink, n_heads)
+    _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)      # float32 [far + 1, heads]: added to the scaled score of a key n positions back
     if qkv.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16:
         raise KernelError("attention_decode: bfloat16 tensors")
@@ -461,14 +518,14 @@ def attention_decode(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
     _contig("qkv", qkv), _contig("out", out), _contig("cache", cache), _contig("block_table", block_table)
     f = _fn("attn_decode", "il_attn_decode", [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int,
                                               _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_void_p,
-                                              _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p],
+                                              _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p],
             defines={"HEAD_DIM": head_dim})
     if kv_map is not None and (kv_map.is_cuda or kv_map.dtype != torch.uint8 or kv_map.numel() != KV_MAP_BYTES):
         raise KernelError("attention_decode: kv_map must be the host tensor kv_tensor_map returned")
     _check(f(_ptr(qkv), qkv.shape[1], _ptr(out), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(entry_kvlen),
              page_size, n_decode, n_heads, n_kv_heads, head_dim, scale, int(window or 0), pages_per_split, n_splits,
              _ptr(o_part), _ptr(ml_part), _ptr(kv_map), _ptr(stream_status(qkv.device)) if kv_map is not None else _c_void_p(0),
-             _ptr(sink), 1 if v_is_k else 0, _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, _stream()), "attention_decode")
+             _ptr(sink), 1 if v_is_k else 0, _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), _stream()), "attention_decode")
     if n_splits > 1:
         count_launches(1)                         # the merge kernel (a single split needs none: the attention kernel finishes the rows)
 
@@ -514,11 +571,12 @@ def kv_tensor_map(cache: torch.Tensor) -> Optional[torch.Tensor]:
 def attention_prefill(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                       entry_qstart: torch.Tensor, entry_kvlen: torch.Tensor, first_entry: int, n_entries: int,
                       n_tiles_total: int, page_size: int, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
-                      window: Optional[int], sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None) -> None:
+                      window: Optional[int], sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
+                      sigmoid: bool = False) -> None:
     """bfloat16 causal attention of the tokens of entries [first_entry, n_entries) over their cache pages.
     n_tiles_total = sum over those entries of ceil(q_len / (64 // (heads/kv_heads)))."""
     _need_cuda(qkv, out, cache, block_table, entry_qstart, entry_kvlen, sink, dist_bias)
-    _check_sink(sink, n_heads)
+    _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)
     if qkv.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16:
         raise KernelError("attention_prefill: bfloat16 tensors")
@@ -527,10 +585,10 @@ def attention_prefill(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor,
     _contig("qkv", qkv), _contig("out", out), _contig("cache", cache), _contig("block_table", block_table)
     f = _fn("attn_prefill", "il_attn_prefill", [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p,
                                                 _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
-                                                _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p], defines={"HEAD_DIM": head_dim})
+                                                _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p], defines={"HEAD_DIM": head_dim})
     _check(f(_ptr(qkv), qkv.shape[1], _ptr(out), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(entry_qstart),
              _ptr(entry_kvlen), page_size, first_entry, n_entries, n_tiles_total, n_heads, n_kv_heads, head_dim, scale,
-             int(window or 0), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, _stream()), "attention_prefill")
+             int(window or 0), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), _stream()), "attention_prefill")
 
 
 _tc5_prefill_rows = {}
@@ -568,11 +626,12 @@ def _has_third_map(kv_map: torch.Tensor) -> bool:
 def attention_prefill_tc5(qkv: torch.Tensor, out: torch.Tensor, kv_map: torch.Tensor, block_table: torch.Tensor,
                           entry_qstart: torch.Tensor, entry_kvlen: torch.Tensor, first_entry: int, n_entries: int,
                           n_tiles_total: int, page_size: int, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
-                          window: Optional[int], sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None) -> None:
+                          window: Optional[int], sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
+                          sigmoid: bool = False) -> None:
     """The same attention as `attention_prefill`, on tcgen05 tensor cores with tensor memory; `kv_map` is the cache's
     tensor map (`kv_tensor_map`). n_tiles_total = sum over the entries of ceil(q_len / (prefill_tc5_rows(head_dim) // (heads/kv_heads)))."""
     _need_cuda(qkv, out, block_table, entry_qstart, entry_kvlen, sink, dist_bias)
-    _check_sink(sink, n_heads)
+    _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)
     if qkv.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("attention_prefill_tc5: bfloat16 tensors")
@@ -583,11 +642,11 @@ def attention_prefill_tc5(qkv: torch.Tensor, out: torch.Tensor, kv_map: torch.Te
     _contig("qkv", qkv), _contig("out", out), _contig("block_table", block_table)
     f = _fn("attn_prefill_tc5", "il_attn_prefill_tc5",
             [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p], defines={"HEAD_DIM": head_dim})
+             _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p], defines={"HEAD_DIM": head_dim})
     _check(f(_ptr(qkv), qkv.shape[1], _ptr(out), _c_void_p(kv_map.data_ptr() + 256), _ptr(block_table), block_table.shape[1],
              _ptr(entry_qstart), _ptr(entry_kvlen), page_size, first_entry, n_entries, n_tiles_total, n_heads, n_kv_heads,
              head_dim, scale, int(window or 0), _ptr(stream_status(qkv.device)), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1,
-             _stream()), "attention_prefill_tc5")
+             int(sigmoid), _stream()), "attention_prefill_tc5")
 
 
 SKINNY_MAX_ROWS = 16
@@ -600,6 +659,16 @@ class ResidualCopy:
 
     def __init__(self, rows: torch.Tensor):
         self.rows = rows
+
+
+class StreamDone:
+    """What a block hands the next when its branches are in the residual stream already: nothing is pending, and `normed`, if
+    not None, holds the next block's first normed input (made with that block's own norm)."""
+    __slots__ = ("normed",)
+    nothing_pending = True
+
+    def __init__(self, normed: Optional[torch.Tensor] = None):
+        self.normed = normed
 
 
 class StreamSet:
@@ -640,9 +709,9 @@ def _norm_args(norm_in: Optional[NormedInput], M: int):
 
 
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, alpha: float = 1.0,
-                bias: Optional[torch.Tensor] = None, glu: int = 0, norm_in: Optional[NormedInput] = None) -> None:
+                bias: Optional[torch.Tensor] = None, glu: int = 0, norm_in: Optional[NormedInput] = None, act_params=None) -> None:
     """out[M,N] = alpha * x[M,K] @ w[N,K]^T (+ bias) for M <= 16 bfloat16 rows; out bfloat16 or float32.
-    glu (True, or ACT_SILU / ACT_GELU_TANH): w is [2N,K] (gate rows, then up rows) and out[M,N] = act(gate) * up.
+    glu (True, or ACT_SILU / ACT_GELU_TANH / ACT_CLAMPED with act_params): w is [2N,K] (gate rows, then up rows) and out[M,N] = act(gate) * up.
     norm_in: x is `norm_in.xw`, and the results are divided by the rms that its sums give."""
     _need_cuda(x, w, out, bias)
     M, K = x.shape
@@ -655,10 +724,11 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, alpha: floa
         raise KernelError("gemm_skinny: bias float32, one per weight row")
     f = _fn("gemm_skinny", "il_gemm_skinny", [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p,
                                               _c_float, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_float,
-                                              _c_void_p])
+                                              _c_float, _c_float, _c_void_p])
+    limit, act_alpha = _act_args(glu, act_params)
     np_, nb, nw, ne = _norm_args(norm_in, M)
     _check(f(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(out), kind_of(out.dtype), out.stride(0), _ptr(bias), alpha,
-             M, N, K, int(glu), np_, nb, nw, ne, _stream()), "gemm_skinny")
+             M, N, K, int(glu), np_, nb, nw, ne, limit, act_alpha, _stream()), "gemm_skinny")
 
 
 def skinny_resid_ok(M: int, K: int, width: int) -> bool:
@@ -808,10 +878,10 @@ def mid_ok(M: int, K: int) -> bool:
 
 
 def gemm_mid(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, alpha: float = 1.0, bias: Optional[torch.Tensor] = None,
-             glu: int = 0, nb: int = 0, bm: int = 0) -> None:
+             glu: int = 0, nb: int = 0, bm: int = 0, act_params=None) -> None:
     """out[M,N] = alpha * x[M,K] @ w[N,K]^T (+ bias) for 17..128 bfloat16 rows on the tcgen05 tensor cores: tiles of 64
     or 128 weight rows (`bm`; the A operand) by blocks of `nb` activation rows (0: chosen by the kernel) over all of K; out bfloat16
-    or float32. glu (True, or ACT_SILU / ACT_GELU_TANH): w is [2N,K] (gate rows, then up rows) and out[M,N] = act(gate) * up (bfloat16)."""
+    or float32. glu (True, or ACT_SILU / ACT_GELU_TANH / ACT_CLAMPED with act_params): w is [2N,K] (gate rows, then up rows) and out[M,N] = act(gate) * up (bfloat16)."""
     _need_cuda(x, w, out, bias)
     M, K = x.shape
     N = w.shape[0] // 2 if glu else w.shape[0]
@@ -822,9 +892,10 @@ def gemm_mid(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, alpha: float =
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != w.shape[0]):
         raise KernelError("gemm_mid: bias float32, one per weight row")
     f = _fn("gemm_mid", "il_gemm_mid", [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_float,
-                                        _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p])
+                                        _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p, _c_void_p])
+    limit, act_alpha = _act_args(glu, act_params)
     _check(f(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(out), kind_of(out.dtype), out.stride(0), _ptr(bias), alpha,
-             M, N, K, int(glu), nb, bm, _ptr(stream_status(x.device)), _stream()), "gemm_mid")
+             M, N, K, int(glu), nb, bm, limit, act_alpha, _ptr(stream_status(x.device)), _stream()), "gemm_mid")
 
 
 _c_ll = ctypes.c_longlong
@@ -891,6 +962,40 @@ def latent_norm_store(proj: torch.Tensor, off_a: int, n_a: int, off_b: int, n_b:
              T, _stream()), "latent_norm_store")
 
 
+def latent_rope_store(proj: torch.Tensor, off_q: int, n_heads: int, q_dim: int, off_b: int, n_b: int, rot_part: int, head_dim: int,
+                      w_b: torch.Tensor, eps: float, rot_dim: int, freq: Optional[torch.Tensor], mscale: float, interleaved: bool,
+                      q_out: torch.Tensor, tok_pos: torch.Tensor, tok_entry: torch.Tensor, block_table: torch.Tensor,
+                      cache: Optional[torch.Tensor], page_size: int) -> None:
+    """Per row of `proj`: columns [off_b, off_b + n_b) are divided by their root mean square and multiplied by `w_b`; the
+    `rot_part` columns behind them turn by pos * freq (their first rot_dim dimensions; `freq` float64 [rot_dim / 2]; cosine and
+    sine times mscale; pairs (2i, 2i + 1) if `interleaved`, else (i, i + rot_dim / 2)); both, with zeros up to head_dim, go to
+    the token's slot of `cache` [pages, 2, 1, page, head_dim], K plane and V plane alike. Head j's query stands at
+    off_q + j * (q_dim + rot_part); its last rot_part columns turn likewise into q_out[t, j * head_dim + n_b ..] (zeros
+    behind), q_out [T, heads * head_dim]; the first n_b columns of a head of q_out are left alone."""
+    _need_cuda(proj, w_b, freq, q_out, tok_pos, tok_entry, block_table, cache)
+    T = proj.shape[0]
+    if proj.stride(1) != 1 or off_q + n_heads * (q_dim + rot_part) > proj.shape[1] or off_b + n_b + rot_part > proj.shape[1]:
+        raise KernelError("latent_rope_store: segments lie outside the rows")
+    if w_b.numel() != n_b or tuple(q_out.shape) != (T, n_heads * head_dim) or q_out.dtype != proj.dtype or not q_out.is_contiguous():
+        raise KernelError("latent_rope_store: w_b [n_b], q_out [T, heads * head_dim] of proj's dtype")
+    if head_dim < n_b + rot_part or rot_dim % 2 or not 0 <= rot_dim <= rot_part:
+        raise KernelError("latent_rope_store: head_dim >= n_b + rot_part, rot_dim even and at most rot_part")
+    if rot_dim and (freq is None or freq.dtype != torch.float64 or freq.numel() != rot_dim // 2):
+        raise KernelError("latent_rope_store: freq float64 [rot_dim / 2]")
+    _i32("latent_rope_store", tok_pos, tok_entry, block_table)
+    _contig("block_table", block_table)
+    if cache is not None:
+        _contig("cache", cache)
+        if cache.dtype != proj.dtype or tuple(cache.shape[1:]) != (2, 1, page_size, head_dim):
+            raise KernelError("latent_rope_store: cache [pages,2,1,page,head_dim] of proj's dtype")
+    f = _fn("latent", "il_latent_rope_store", [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int,
+                                               _c_float, _c_int, _c_void_p, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
+                                               _c_void_p, _c_int, _c_int, _c_void_p])
+    _check(f(_ptr(proj), kind_of(proj.dtype), proj.stride(0), off_q, n_heads, q_dim, off_b, n_b, rot_part, head_dim, _ptr(w_b),
+             kind_of(w_b.dtype), eps, rot_dim, _ptr(freq if rot_dim else None), mscale, int(interleaved), _ptr(q_out), _ptr(tok_pos),
+             _ptr(tok_entry), _ptr(block_table), block_table.shape[1], _ptr(cache), page_size, T, _stream()), "latent_rope_store")
+
+
 def sigmoid_gate(y: torch.Tensor, gate: torch.Tensor) -> None:
     """y[t, :] *= sigmoid(gate[t, :]) in place; y [T, n] contiguous, gate [T, n] with any row stride, one dtype."""
     _need_cuda(y, gate)
@@ -902,7 +1007,7 @@ def sigmoid_gate(y: torch.Tensor, gate: torch.Tensor) -> None:
 
 
 MOE_MAX_TOP = 32
-ROUTE_TOP_LOGITS, ROUTE_SOFTMAX_ALL = 0, 1         # how a router's logits become choices and weights (`moe_select`)
+ROUTE_TOP_LOGITS, ROUTE_SOFTMAX_ALL, ROUTE_SIGMOID = 0, 1, 2      # how a router's logits become choices and weights (`moe_select`)
 
 
 def moe_route(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], idx: torch.Tensor, wt: torch.Tensor, top: int,
@@ -937,13 +1042,14 @@ def moe_route(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], id
 def moe_route_sort_small(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], z: torch.Tensor, idx: torch.Tensor, wt: torch.Tensor,
                          top: int, group_off: torch.Tensor, pos_of_slot: torch.Tensor, row_of_pos: torch.Tensor,
                          norm_in: Optional["NormedInput"] = None, rstd_out: Optional[torch.Tensor] = None, extra: int = 0,
-                         rule: int = ROUTE_TOP_LOGITS, out_scale: float = 1.0) -> None:
+                         rule: int = ROUTE_TOP_LOGITS, out_scale: float = 1.0, wt_of_pos: Optional[torch.Tensor] = None) -> None:
     """`moe_route` and `moe_sort` for a few bfloat16 rows (a decode step) as two short kernels: the logits, a warp per
     (token, expert), into z [T, E + extra] float32; then one block that chooses for every token and sorts the slots.
     Rows of whole 16-byte chunks (H a multiple of 8); `route_sort_small_ok` says whether a shape is taken.
     `extra`: the last rows of `w` are no experts - their products are written to z's last columns and take no part in the
-    choice. `rule`, `out_scale`: see `moe_select`."""
-    _need_cuda(x, w, bias, z, idx, wt, group_off, pos_of_slot, row_of_pos, rstd_out)
+    choice. `rule`, `out_scale`: see `moe_select`; `wt_of_pos`: see `moe_sort`."""
+    _need_cuda(x, w, bias, z, idx, wt, group_off, pos_of_slot, row_of_pos, rstd_out, wt_of_pos)
+    _check_wt_of_pos("moe_route_sort_small", wt_of_pos, x.shape[0] * top)
     T, H = x.shape
     E = w.shape[0] - extra
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != H or x.stride(1) != 1 or not w.is_contiguous():
@@ -967,10 +1073,10 @@ def moe_route_sort_small(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.
     sq, n_partial, _, eps = _norm_args(norm_in, T)
     f = _fn("moe", "il_moe_route_sort_small", [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
                                                _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
-                                               _c_int, _c_float, _c_void_p])
+                                               _c_int, _c_float, _c_void_p, _c_void_p])
     _check(f(_ptr(x), x.stride(0), _ptr(w), _ptr(bias), kind_of(bias.dtype) if bias is not None else 0, _ptr(z), _ptr(idx), _ptr(wt), T, H, E,
              top, sq, n_partial, eps, _ptr(rstd_out), _ptr(group_off), _ptr(pos_of_slot), _ptr(row_of_pos), int(extra), int(rule),
-             float(out_scale), _stream()), "moe_route_sort_small")
+             float(out_scale), _ptr(wt_of_pos), _stream()), "moe_route_sort_small")
     count_launches(1)                             # two kernels
 
 
@@ -985,7 +1091,9 @@ def moe_select(z: torch.Tensor, bias: Optional[torch.Tensor], idx: torch.Tensor,
     """The choice of `moe_route` for logits a matrix product has written: z [T, E] float32 (+ bias [E]) -> idx, wt [T, top].
     rule ROUTE_TOP_LOGITS: the `top` largest of z + bias, their weights the softmax over the chosen alone.
     rule ROUTE_SOFTMAX_ALL: scores s = softmax(z) over all E; the `top` largest of s + bias are chosen (the lower expert wins a
-    tie); the weights are the chosen experts' s over their sum (+ 1e-20), times out_scale."""
+    tie); the weights are the chosen experts' s over their sum (+ 1e-20), times out_scale.
+    rule ROUTE_SIGMOID: scores s = sigmoid(z); the `top` largest of s + bias are chosen (without a bias: of z, the same order);
+    the weights are the chosen s themselves, times out_scale."""
     _need_cuda(z, bias, idx, wt)
     T, E = z.shape
     if z.dtype != torch.float32 or z.stride(1) != 1:
@@ -1003,17 +1111,29 @@ def moe_select(z: torch.Tensor, bias: Optional[torch.Tensor], idx: torch.Tensor,
              float(out_scale), _stream()), "moe_select")
 
 
-def moe_sort(idx: torch.Tensor, n_experts: int, group_off: torch.Tensor, pos_of_slot: torch.Tensor, row_of_pos: torch.Tensor) -> None:
-    """Orders the slots (token, choice) of idx [T, top] by expert: group_off [E + 1], pos_of_slot [T * top], row_of_pos [T * top]."""
-    _need_cuda(idx, group_off, pos_of_slot, row_of_pos)
+def _check_wt_of_pos(what: str, t: Optional[torch.Tensor], n: int) -> None:
+    if t is not None and (t.dtype != torch.float32 or t.numel() < n or not t.is_contiguous()):
+        raise KernelError(f"{what}: wt_of_pos float32 [T * top], contiguous")
+
+
+def moe_sort(idx: torch.Tensor, n_experts: int, group_off: torch.Tensor, pos_of_slot: torch.Tensor, row_of_pos: torch.Tensor,
+             wt: Optional[torch.Tensor] = None, wt_of_pos: Optional[torch.Tensor] = None) -> None:
+    """Orders the slots (token, choice) of idx [T, top] by expert: group_off [E + 1], pos_of_slot [T * top], row_of_pos [T * top].
+    With `wt` [T, top] and `wt_of_pos` [T * top] (float32) the weights are put into the sorted order too: a factor per place for
+    the products, where a choice's weight belongs to its expert's input."""
+    _need_cuda(idx, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos)
+    _check_wt_of_pos("moe_sort", wt_of_pos, idx.numel())
+    if wt_of_pos is not None and (wt is None or wt.dtype != torch.float32 or wt.numel() != idx.numel() or not wt.is_contiguous()):
+        raise KernelError("moe_sort: wt float32 [T, top] comes with wt_of_pos")
     T, top = idx.shape
     for t in (idx, group_off, pos_of_slot, row_of_pos):
         if t.dtype != torch.int32 or not t.is_contiguous():
             raise KernelError("moe_sort: contiguous int32 tensors")
     if group_off.numel() < n_experts + 1 or pos_of_slot.numel() < T * top or row_of_pos.numel() < T * top:
         raise KernelError("moe_sort: outputs too small")
-    f = _fn("moe", "il_moe_sort", [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p])
-    _check(f(_ptr(idx), T * top, top, n_experts, _ptr(group_off), _ptr(pos_of_slot), _ptr(row_of_pos), _stream()), "moe_sort")
+    f = _fn("moe", "il_moe_sort", [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p])
+    _check(f(_ptr(idx), T * top, top, n_experts, _ptr(group_off), _ptr(pos_of_slot), _ptr(row_of_pos),
+             _ptr(wt if wt_of_pos is not None else None), _ptr(wt_of_pos), _stream()), "moe_sort")
 
 
 def gather_rows(x: torch.Tensor, rows: torch.Tensor, out: torch.Tensor) -> None:
@@ -1027,16 +1147,19 @@ def gather_rows(x: torch.Tensor, rows: torch.Tensor, out: torch.Tensor) -> None:
     _check(f(_ptr(x), kind_of(x.dtype), x.stride(0), _ptr(rows), _ptr(out), n, H, _stream()), "gather_rows")
 
 
-def moe_combine(y: torch.Tensor, pos_of_slot: torch.Tensor, wt: torch.Tensor, shared_rows: Optional[torch.Tensor], out: torch.Tensor, *,
+def moe_combine(y: torch.Tensor, pos_of_slot: torch.Tensor, wt: Optional[torch.Tensor], shared_rows: Optional[torch.Tensor], out: torch.Tensor, *,
                 group_off: Optional[torch.Tensor] = None, n_real: int = 0, x: Optional[torch.Tensor] = None,
-                shared_gate: Optional[torch.Tensor] = None) -> None:
-    """out[t] = sum_k wt[t,k] * y[pos_of_slot[t*top + k]] (+ shared_rows[t]), summed in f32 in the order of k.
+                shared_gate: Optional[torch.Tensor] = None, top: int = 0) -> None:
+    """out[t] = sum_k wt[t,k] * y[pos_of_slot[t*top + k]] (+ shared_rows[t]), summed in f32 in the order of k. wt None (then
+    `top` says how many choices a token has): a plain sum.
     With `group_off` (int32, the sorted order's group starts), `n_real` and `x` [T, H]: the experts from n_real on have no
     weights and return their input - a choice whose place is group_off[n_real] or later adds wt * x[t] instead of a row of y.
     `shared_gate`: float32 [T] (any stride) - the shared row is multiplied by its sigmoid."""
     _need_cuda(y, pos_of_slot, wt, shared_rows, out, group_off, x, shared_gate)
-    T, top = wt.shape
+    T, top = wt.shape if wt is not None else (out.shape[0], int(top))
     H = out.shape[1]
+    if top < 1 or pos_of_slot.numel() < T * top:
+        raise KernelError("moe_combine: pos_of_slot [T * top]")
     if group_off is not None and (x is None or x.dtype != out.dtype or tuple(x.shape) != (T, H) or x.stride(1) != 1
                                   or group_off.dtype != torch.int32 or group_off.numel() <= n_real):
         raise KernelError("moe_combine: identity experts need group_off int32 [> n_real] and x [T, H] of out's dtype")
@@ -1046,7 +1169,9 @@ def moe_combine(y: torch.Tensor, pos_of_slot: torch.Tensor, wt: torch.Tensor, sh
         raise KernelError("moe_combine: y [T * top, H], out [T, H] of the same dtype")
     if shared_rows is not None and (shared_rows.dtype != out.dtype or tuple(shared_rows.shape) != (T, H)):
         raise KernelError("moe_combine: shared_rows [T, H]")
-    _contig("y", y), _contig("out", out), _contig("wt", wt)
+    _contig("y", y), _contig("out", out)
+    if wt is not None:
+        _contig("wt", wt)
     if shared_rows is not None:
         _contig("shared_rows", shared_rows)
     f = _fn("moe", "il_moe_combine", [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int,
@@ -1085,18 +1210,19 @@ def moe_combine_resid(y: torch.Tensor, pos_of_slot: torch.Tensor, wt: torch.Tens
 
 def gemm_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, group_off: Optional[torch.Tensor] = None,
                  a_rows: Optional[torch.Tensor] = None, n_rows: Optional[int] = None, glu: bool = False,
-                 gate: Optional[torch.Tensor] = None, row_scale: Optional[torch.Tensor] = None) -> None:
+                 gate: Optional[torch.Tensor] = None, row_scale: Optional[torch.Tensor] = None, scale_by_place: bool = False) -> None:
     """Products over groups, out_g = a_g w_g^T, w [G, N, K] (glu: [G, 2N, K], gate rows then up rows, out = silu(gate) * up).
     Ragged (`group_off` int32 [G + 1] on the device): the `n_rows` rows of `out` [n_rows, N] stand sorted by group, group g
     owning places group_off[g] .. group_off[g+1] - 1; the row of `a` [*, K] at a place is a_rows[place] (or the place).
     Batched (no `group_off`): a [M, G, K] and out [M, G, N] are column ranges of shared rows; `gate` [M, G, N] multiplies
-    out by its sigmoid.
-    row_scale (ragged, bfloat16 rows of 16-byte chunks): float32 per row of `a`; the products of a row are multiplied by
-    its factor before the epilogue (the rstd of a norm the rows have not been divided by)."""
+    out by its sigmoid; a gate [M, G] is one number per group and row.
+    row_scale (ragged): float32 per row of `a` - or, with scale_by_place, per place of the sorted order; the products of a row
+    are multiplied by its factor before the epilogue (the rstd of a norm the rows have not been divided by; the weight of a
+    choice that belongs to its expert's input)."""
     _need_cuda(a, w, out, group_off, a_rows, gate, row_scale)
     if row_scale is not None and (group_off is None or row_scale.dtype != torch.float32 or not row_scale.is_contiguous()
-                                  or row_scale.numel() < a.shape[0]):
-        raise KernelError("gemm_grouped: row_scale float32 [rows of a], with the ragged form")
+                                  or row_scale.numel() < (int(n_rows if n_rows is not None else out.shape[0]) if scale_by_place else a.shape[0])):
+        raise KernelError("gemm_grouped: row_scale float32 [rows of a] (scale_by_place: [places]), with the ragged form")
     if w.dim() != 3 or not w.is_contiguous() or w.dtype != a.dtype or out.dtype != a.dtype:
         raise KernelError("gemm_grouped: w [G, N, K] contiguous, one dtype for a, w and out")
     G, K = w.shape[0], w.shape[2]
@@ -1111,7 +1237,7 @@ def gemm_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, group_o
             raise KernelError("gemm_grouped: a has fewer rows than places")
         if gate is not None:
             raise KernelError("gemm_grouped: gate goes with the batched form")
-        lda, a_gs, ldc, c_gs, ldg, g_gs = a.stride(0), 0, out.stride(0), 0, 0, 0
+        lda, a_gs, ldc, c_gs, ldg, g_gs, g_ns = a.stride(0), 0, out.stride(0), 0, 0, 0, 1
     else:
         if a.dim() != 3 or out.dim() != 3 or a.shape[1] != G or out.shape[1] != G or a.shape[2] != K or out.shape[2] != N or a.shape[0] != out.shape[0]:
             raise KernelError(f"gemm_grouped: batched a{tuple(a.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
@@ -1119,16 +1245,20 @@ def gemm_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, group_o
             raise KernelError("gemm_grouped: innermost dimension must be contiguous")
         M = a.shape[0]
         lda, a_gs, ldc, c_gs = a.stride(0), a.stride(1), out.stride(0), out.stride(1)
-        ldg = g_gs = 0
-        if gate is not None:
+        ldg, g_gs, g_ns = 0, 0, 1
+        if gate is not None and gate.dim() == 2:
+            if tuple(gate.shape) != (M, G) or gate.dtype != out.dtype:
+                raise KernelError("gemm_grouped: a gate per group is [M, G] of out's dtype")
+            ldg, g_gs, g_ns = gate.stride(0), gate.stride(1), 0
+        elif gate is not None:
             if tuple(gate.shape) != tuple(out.shape) or gate.dtype != out.dtype or gate.stride(2) != 1:
                 raise KernelError("gemm_grouped: gate [M, G, N] of out's dtype")
             ldg, g_gs = gate.stride(0), gate.stride(1)
     f = _fn("gemm_grouped", "il_gemm_grouped", [_c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_void_p, _c_int, _c_ll, _c_void_p, _c_int,
                                                 _c_ll, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_ll,
-                                                _c_void_p, _c_void_p])
+                                                _c_int, _c_void_p, _c_int, _c_void_p])
     _check(f(_ptr(a), kind_of(a.dtype), lda, a_gs, _ptr(a_rows), _ptr(w), w.stride(1), w.stride(0), _ptr(out), ldc, c_gs, _ptr(group_off),
-             G, M, N, K, int(glu), _ptr(gate), ldg, g_gs, _ptr(row_scale), _stream()), "gemm_grouped")
+             G, M, N, K, int(glu), _ptr(gate), ldg, g_gs, g_ns, _ptr(row_scale), int(scale_by_place), _stream()), "gemm_grouped")
 
 
 # ----------------------------------------------------------------------------------------------

@@ -31,7 +31,8 @@ class PagedAttend:
     positions back as dist_bias[min(n, far), head] (constant from `far` on).
     `chunk`: instead of a sliding window, runs of `chunk` positions counted from position 0 of the sequence; a query sees the
     keys of its own run up to itself (the kernels take it as a negative window). The cache keeps every page: a window's
-    pages are given back behind it, a chunked layer's are not (another layer may read them)."""
+    pages are given back behind it, a chunked layer's are not (another layer may read them).
+    `sigmoid`: no softmax - a visible key's weight is the sigmoid of its score (scaled, biased), not normalised over the keys."""
 
     # The fast bfloat16 kernels take kernel pages of 16 keys (the cache manager lays larger pages out as runs of them)
     # and at most 64 query heads per kv head; anything else, and the whole float32 path, runs the plain kernel.
@@ -42,7 +43,8 @@ class PagedAttend:
     WAVE_FILL = 2.0 / 3.0                         # share of the blocks the device holds at once that the splits aim at
 
     def __init__(self, dtype, n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: Optional[int] = None,
-                 force_plain: bool = False, prefill_kernel: str = "auto", shared_kv: bool = False, chunk: Optional[int] = None):
+                 force_plain: bool = False, prefill_kernel: str = "auto", shared_kv: bool = False, chunk: Optional[int] = None,
+                 sigmoid: bool = False):
         if chunk is not None and (window is not None or int(chunk) < 1):
             raise ValueError("attention: a mask is a window or runs of a positive size, not both")
         self.dtype, self.nh, self.nkv, self.hd, self.scale, self.window = dtype, n_heads, n_kv_heads, head_dim, scale, window
@@ -50,6 +52,7 @@ class PagedAttend:
         self.span = self.chunk if self.chunk is not None else window          # the most keys a query sees (None: all)
         self.mask_arg = -self.chunk if self.chunk is not None else window     # what the kernels take
         self.force_plain, self.prefill_kernel, self.shared_kv = force_plain, prefill_kernel, shared_kv
+        self.sigmoid = bool(sigmoid)
         self.sink: Optional[torch.Tensor] = None
         self.dist_bias: Optional[torch.Tensor] = None
 
@@ -74,7 +77,7 @@ class PagedAttend:
                               "head sizes in steps of 16 up to 256): the plain kernel runs, at a fraction of their speed",
                               RuntimeWarning, stacklevel=2)
             ops.attention_plain(qkv, out, cache.storage, cache.block_table, ctx.tok_pos, ctx.tok_entry,
-                                cache.page_size, self.nh, self.nkv, self.hd, self.scale, self.mask_arg, self.sink, self.dist_bias)
+                                cache.page_size, self.nh, self.nkv, self.hd, self.scale, self.mask_arg, self.sink, self.dist_bias, self.sigmoid)
             return
         n_dec, E = ctx.n_decode, ctx.n_entries
         if n_dec > 0:
@@ -90,7 +93,7 @@ class PagedAttend:
                                  self.nh, self.nkv, self.hd, self.scale, self.mask_arg, 0, n_splits,
                                  ctx.ws.flat("attn_o_part", rows * self.hd, torch.float32),
                                  ctx.ws.flat("attn_ml_part", rows * 2, torch.float32), kv_map=cache.tma_map, sink=self.sink,
-                                 v_is_k=v_is_k, dist_bias=self.dist_bias)
+                                 v_is_k=v_is_k, dist_bias=self.dist_bias, sigmoid=self.sigmoid)
         if E > n_dec:
             # prompt portions: on tcgen05 with tensor memory where the head size has that kernel (64, 128, 256) and the cache
             # its tensor map; else the mma.sync kernel. The tile is 128 (64) rows = tokens x heads of a kv head.
@@ -101,11 +104,11 @@ class PagedAttend:
             if tc5:
                 ops.attention_prefill_tc5(qkv, out, cache.tma_map, cache.block_table, ctx.entry_qstart, ctx.entry_kvlen,
                                           n_dec, E, n_tiles, cache.page_size, self.nh, self.nkv, self.hd, self.scale,
-                                          self.mask_arg, sink=self.sink, dist_bias=self.dist_bias)
+                                          self.mask_arg, sink=self.sink, dist_bias=self.dist_bias, sigmoid=self.sigmoid)
             else:
                 ops.attention_prefill(qkv, out, cache.storage, cache.block_table, ctx.entry_qstart, ctx.entry_kvlen,
                                       n_dec, E, n_tiles, cache.page_size, self.nh, self.nkv, self.hd, self.scale,
-                                      self.mask_arg, sink=self.sink, dist_bias=self.dist_bias)
+                                      self.mask_arg, sink=self.sink, dist_bias=self.dist_bias, sigmoid=self.sigmoid)
 
 
 class Attention(Mixer):
@@ -134,6 +137,8 @@ class Attention(Mixer):
         self.position = build_part("position", pos, dtype)
         if self.position.rot_dim > self.hd:
             raise ValueError("attention: rotary dim exceeds head_dim")
+        if self.position.interleaved:
+            raise ValueError("attention: its rotary table pairs dimension i with i + rot_dim / 2")
         if self.position.has_transform and self.position.rot_dim:
             raise ValueError("attention: a position encoding is a rotary table or a transform, not both")
 

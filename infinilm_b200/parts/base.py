@@ -68,7 +68,7 @@ class PositionEncoding(Part):
     """A position encoding that a mixer applies to its queries and keys. Two forms:
 
     rotary: `rot_dim`, `inv_freq`, `mscale` - a table that the mixer's fused rotate-and-store kernel applies
-      (angle = position * inv_freq[i], pairs (i, i + rot_dim/2), cos and sin times mscale);
+      (angle = position * inv_freq[i], pairs (i, i + rot_dim/2) - or (2i, 2i + 1) where `interleaved` -, cos and sin times mscale);
     any other function of (q, k, position): `has_transform = True` and `transform(qkv, ctx, ...)`, which changes the
       q and k columns of the projected rows in place before the keys are written to the cache (rot_dim stays 0). The
       mixer then leaves its fused projection-and-rotation kernel for the plain sequence projection, transform, store.
@@ -76,6 +76,8 @@ class PositionEncoding(Part):
     rot_dim: int = 0
     mscale: float = 1.0
     inv_freq: Optional[torch.Tensor] = None     # float32 [rot_dim/2] on the device
+    freq64: Optional[torch.Tensor] = None       # the same in float64, for a kernel that makes its angles in double precision
+    interleaved = False                         # True: dimension 2i turns with 2i + 1 (a mixer that cannot pair so refuses the encoding)
     has_transform = False
 
     def to_device(self, device: torch.device) -> None:
@@ -116,6 +118,9 @@ class FeedForward(Part):
 
     def fuses_tail(self, T: int) -> bool:
         return False
+
+    # True: `forward(x, ctx, routed=True)` returns an `ops.RoutedRows` for a reader that sums a token's rows itself
+    gives_routed_rows = False
 
 
 class Arrangement:

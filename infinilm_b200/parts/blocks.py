@@ -14,7 +14,7 @@ from typing import Dict, List
 import torch
 
 from .. import ops
-from .base import Arrangement, Part, ResidualTail, register_part
+from .base import Arrangement, Part, ResidualTail, build_part, register_part
 from .spec import WeightSpec
 
 
@@ -105,6 +105,46 @@ class BranchNormResidual(Arrangement):
         return ops.ResidualCopy(x)
 
 
+class SandwichResidual(Arrangement):
+    """h += norm_b1(mixer(norm1(h))); h += norm_b2(ffn(norm2(h))): a norm in front of every sublayer and one on its output,
+    before it joins the stream. params: mixer_branch_norm, ffn_branch_norm (PartSpecs of RMS norms). One kernel does what lies
+    between two sublayers - the norm of the branch (and, behind a routed feed-forward, the sum over a token's rows), the add, the
+    next norm - also across the border to the next block of this kind. (The statistics of a branch's norm are those of the
+    product's whole output row, so unlike a norm in front of a product it cannot move into the product before it.)"""
+
+    takes_next_block = True
+
+    def __init__(self, mixer_norm, mixer, ffn_norm, ffn, params):
+        super().__init__(mixer_norm, mixer, ffn_norm, ffn, params)
+        self.mixer_branch_norm = build_part("norm", params["mixer_branch_norm"], mixer_norm.dtype)
+        self.ffn_branch_norm = None if ffn is None else build_part("norm", params["ffn_branch_norm"], mixer_norm.dtype)
+        if not all(n is None or n.fusable_rms for n in (mixer_norm, ffn_norm, self.mixer_branch_norm, self.ffn_branch_norm)):
+            raise ValueError("a block with norms on both sides of its sublayers takes RMS norms")
+
+    def parts(self):
+        return super().parts() + [n for n in (self.mixer_branch_norm, self.ffn_branch_norm) if n is not None]
+
+    def run(self, resid, pending, ctx, cache, next_block=None):
+        T, H = resid.shape
+        normed = ctx.ws.rows("normed", T, H, ctx.dtype)
+        if isinstance(pending, ops.NormedInput):
+            raise ValueError("a block with norms on both sides of its sublayers cannot take a half-done norm")
+        if isinstance(pending, ops.StreamDone) and pending.normed is not None:
+            normed = pending.normed
+        else:
+            branch, bscale = pending if isinstance(pending, tuple) else (None, 1.0)
+            self.mixer_norm.add_norm(resid, branch, bscale, normed)
+        branch = self.mixer.forward(normed, ctx, cache)
+        nxt = next_block if isinstance(next_block, SandwichResidual) else None
+        after = self.mixer_branch_norm                # the norm of the branch that has just been computed
+        if self.ffn is not None:
+            after.norm_add_norm(resid, branch, self.ffn_norm, normed)
+            branch = self.ffn.forward(normed, ctx, routed=True) if self.ffn.gives_routed_rows else self.ffn.forward(normed, ctx)
+            after = self.ffn_branch_norm
+        after.norm_add_norm(resid, branch, None if nxt is None else nxt.mixer_norm, normed)
+        return ops.StreamDone(None if nxt is None else normed)
+
+
 class StreamWeights(Part):
     """The numbers by which a block with several copies of the residual stream reads and writes them, per sublayer q (1: the
     mixer, 2: the feed-forward): hc<q>.in [S] (the sublayer's input is sum_s in[s] x_s), hc<q>.mix [S, S] (from, to) and
@@ -192,3 +232,4 @@ class HyperConnections(Arrangement):
 register_part("arrangement", "prenorm_residual", PreNormResidual)
 register_part("arrangement", "hyper_connections", HyperConnections)
 register_part("arrangement", "branch_norm_residual", BranchNormResidual)
+register_part("arrangement", "sandwich_residual", SandwichResidual)

@@ -1,4 +1,5 @@
-"""Dense gated feed-forward: down(act(gate(x)) * up(x)), act SiLU (SwiGLU) or the tanh form of GELU.
+"""Dense gated feed-forward: down(act(gate(x)) * up(x)), act SiLU (SwiGLU) or the tanh form of GELU; or, "clamped", with
+g = min(gate(x), limit) and u = up(x) kept within -limit .. limit: down(g sigmoid(alpha g) (u + 1)).
 
 Parity with InfiniLM: `csrc/layers/mlp/mlp.cpp:7-38` (gate and up as one product, `swiglu(up, gate)`,
 then down), `csrc/layers/linear/fused_linear.cpp:152-158,177-185` (gate rows first, up rows second).
@@ -16,10 +17,11 @@ from .spec import WeightSpec
 
 
 class SwiGLU(FeedForward):
-    """params: hidden, intermediate, bias, out_scale; activation ("silu", the default, or "gelu_tanh": the gate's function);
+    """params: hidden, intermediate, bias, out_scale; activation ("silu", the default, or "gelu_tanh": the gate's function; or
+    "clamped" with limit and alpha);
     names (local tensor names of the three weights, default gate_proj.weight / up_proj.weight / down_proj.weight)."""
     graph_safe = True
-    ACTIVATIONS = {"silu": ops.ACT_SILU, "gelu_tanh": ops.ACT_GELU_TANH}
+    ACTIVATIONS = {"silu": ops.ACT_SILU, "gelu_tanh": ops.ACT_GELU_TANH, "clamped": ops.ACT_CLAMPED}
 
     def __init__(self, params, prefix, dtype):
         super().__init__(params, prefix, dtype)
@@ -29,6 +31,9 @@ class SwiGLU(FeedForward):
         if act not in self.ACTIVATIONS:
             raise ValueError(f"gated feed-forward: activation {act!r} is not one of {', '.join(self.ACTIVATIONS)}")
         self.act = self.ACTIVATIONS[act]
+        self.act_params = (float(params["limit"]), float(params["alpha"])) if self.act == ops.ACT_CLAMPED else None
+        if self.act_params is not None and not self.act_params[0] > 0.0:
+            raise ValueError("gated feed-forward: the clamped gate's limit must be positive")
         names = params.get("names") or {}
         self.n_gate, self.n_up, self.n_down = (str(names.get(k, d)) for k, d in
                                                (("gate", "gate_proj.weight"), ("up", "up_proj.weight"), ("down", "down_proj.weight")))
@@ -63,9 +68,9 @@ class SwiGLU(FeedForward):
             # decode: gate and up rows streamed together, SiLU(gate)*up in the epilogue
             act = ctx.ws.rows("ffn_act", T, self.inter, self.dtype)
             if isinstance(x, ops.NormedInput):
-                ops.gemm_skinny(x.xw, self.gate_up.weight, act, 1.0, self.gate_up.bias, glu=self.act, norm_in=x)
+                ops.gemm_skinny(x.xw, self.gate_up.weight, act, 1.0, self.gate_up.bias, glu=self.act, norm_in=x, act_params=self.act_params)
             else:
-                ops.gemm_skinny(x, self.gate_up.weight, act, 1.0, self.gate_up.bias, glu=self.act)
+                ops.gemm_skinny(x, self.gate_up.weight, act, 1.0, self.gate_up.bias, glu=self.act, act_params=self.act_params)
             if tail is not None:                  # down adds into the residual and prepares the next norm itself
                 return ops.gemm_skinny_resid(act, self.down.weight, self.down.alpha, self.down.bias, tail.resid, tail.scale,
                                              tail.norm.weight, tail.norm.eps,
@@ -77,10 +82,10 @@ class SwiGLU(FeedForward):
             # 17..128 rows: gate and up on the tcgen05 tensor cores as two accumulators in the same lanes, SiLU(gate)*up in
             # the epilogue (measured against the library product followed by the SwiGLU kernel at 8B sizes: 44.6 against
             # 48.4 us at 32 rows, 47.6 against 49.9 at 64, 52.5 against 57.6 at 128)
-            ops.gemm_mid(x, self.gate_up.weight, act, 1.0, self.gate_up.bias, glu=self.act)
+            ops.gemm_mid(x, self.gate_up.weight, act, 1.0, self.gate_up.bias, glu=self.act, act_params=self.act_params)
             return self.down(act, ctx.ws.rows("branch", T, self.hidden, self.dtype))
         gu = self.gate_up(x, ctx.ws.rows("gate_up", T, 2 * self.inter, self.dtype))
-        ops.swiglu(gu, act, self.act)
+        ops.swiglu(gu, act, self.act, self.act_params)
         return self.down(act, ctx.ws.rows("branch", T, self.hidden, self.dtype))
 
 

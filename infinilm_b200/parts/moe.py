@@ -10,6 +10,12 @@ sum (+ 1e-20), times `route_scale`. The router's last `n_identity` outputs may s
 their input (weight_k * h), and the shared unit may be multiplied by sigmoid(w_sg . h), one number per token: that row
 rides along as one more row of the router's product and takes no part in the choice.
 
+A third rule (`route_rule` "sigmoid"): s = sigmoid(z), each output on its own; the `top` largest are chosen and the chosen s are
+the weights as they stand (times `route_scale`). With `weight_on_input` a choice's weight multiplies the row its expert reads,
+unit(weight_k * h), instead of what the expert returns: the sort brings the weights into the order of the sorted rows and
+the gate+up product takes them as a factor per row (a linear map: W (weight h) = weight (W h), without rounding weight h); the
+combine then sums plainly.
+
 Everything stays on the device: the router kernel writes the choices, a sort kernel orders the (token, choice) slots by
 expert, two products over those ragged groups run the experts (gate and up as one product with the SiLU in its
 epilogue, then down), and a combine kernel sums a token's rows in the order of its choices. Nothing is read back, so a
@@ -36,7 +42,7 @@ from .spec import WeightSpec
 
 class RoutedExperts(FeedForward):
     """params: hidden, n_experts (units with weights), top, expert_ff, shared_ff (None: no shared unit), router_bias;
-    route_rule ("top_logits", the default, or "softmax_all"), route_scale, n_identity (router outputs behind the experts' that
+    route_rule ("top_logits", the default, "softmax_all" or "sigmoid"), weight_on_input, route_scale, n_identity (router outputs behind the experts' that
     return the input), shared_gate (the shared unit times the sigmoid of a row `shared.sg` [1, hidden]), bias_name (the tensor
     of the router's per-output numbers: "router.b")."""
     graph_safe = True
@@ -57,15 +63,21 @@ class RoutedExperts(FeedForward):
         self.shared_ff = None if p.get("shared_ff") is None else int(p["shared_ff"])
         self.router_bias = bool(p.get("router_bias", True))
         rule = str(p.get("route_rule", "top_logits"))
-        if rule not in ("top_logits", "softmax_all"):
-            raise ValueError("routed experts: route_rule is 'top_logits' or 'softmax_all'")
-        self.rule = ops.ROUTE_SOFTMAX_ALL if rule == "softmax_all" else ops.ROUTE_TOP_LOGITS
+        rules = {"top_logits": ops.ROUTE_TOP_LOGITS, "softmax_all": ops.ROUTE_SOFTMAX_ALL, "sigmoid": ops.ROUTE_SIGMOID}
+        if rule not in rules:
+            raise ValueError(f"routed experts: route_rule is one of {', '.join(rules)}")
+        self.rule = rules[rule]
+        self.w_on_input = bool(p.get("weight_on_input", False))
         self.route_scale, self.n_id = float(p.get("route_scale", 1.0)), int(p.get("n_identity", 0))
         self.has_sg = bool(p.get("shared_gate", False))
         self.bias_name = str(p.get("bias_name", "router.b"))
         self.n_out = self.n + self.n_id           # the router's outputs: the experts, then the identity units
         # anything beyond the first rule: the logits go through memory (a product, then the choice), never the fused router
-        self.extended = self.rule != ops.ROUTE_TOP_LOGITS or self.n_id > 0 or self.has_sg
+        self.extended = self.rule != ops.ROUTE_TOP_LOGITS or self.n_id > 0 or self.has_sg or self.w_on_input
+        if self.w_on_input and self.n_id > 0:
+            raise ValueError("routed experts: identity units go with weights on the experts' outputs")
+        # the rows of a token's choices can be left to a reader that sums them itself (nothing but the choices is in the branch)
+        self.gives_routed_rows = self.shared_ff is None and self.n_id == 0
         if self.n_id < 0 or (self.has_sg and p.get("shared_ff") is None):
             raise ValueError("routed experts: n_identity >= 0; a shared gate needs a shared unit")
         if not 0 < self.top <= min(self.n_out, ops.MOE_MAX_TOP) or self.n <= 0:
@@ -125,7 +137,7 @@ class RoutedExperts(FeedForward):
         return (self.dtype == torch.bfloat16 and not self.extended and 0 < T <= ops.SKINNY_MAX_ROWS and self.hidden % 4 == 0
                 and (self.hidden + 15) // 16 <= ops.NORM_MAX_BLOCKS)
 
-    def forward(self, x, ctx, tail=None):
+    def forward(self, x, ctx, tail=None, routed=False):
         T, W, k = x.shape[0], self.hidden, self.top
         ws, dt, n_slots = ctx.ws, self.dtype, x.shape[0] * self.top
         idx = ws.rows("moe_idx", T, k, torch.int32)
@@ -134,6 +146,7 @@ class RoutedExperts(FeedForward):
         group_off = ws.flat("moe_group_off", self.n_out + 1, torch.int32)
         pos_of_slot = ws.rows("moe_pos", T, k, torch.int32).view(-1)
         row_of_pos = ws.rows("moe_row", T, k, torch.int32).view(-1)
+        wt_of_pos = ws.rows("moe_wt_place", T, k, torch.float32).view(-1) if self.w_on_input else None
         if isinstance(x, ops.NormedInput):       # x.xw = residual * norm weight; the division by the rms is still to come
             normed_in, rstd = x, ws.flat("moe_rstd", T, torch.float32)
         rows = x if normed_in is None else x.xw
@@ -147,7 +160,7 @@ class RoutedExperts(FeedForward):
             z = ws.rows("moe_logits", T, EZ, torch.float32)
             if small:
                 ops.moe_route_sort_small(rows, self.router, self.router_b, z, idx, wt, k, group_off, pos_of_slot, row_of_pos,
-                                         extra=EZ - self.n_out, rule=self.rule, out_scale=self.route_scale)
+                                         extra=EZ - self.n_out, rule=self.rule, out_scale=self.route_scale, wt_of_pos=wt_of_pos)
             else:
                 self.router_lin(x, z, out_f32=True)
                 ops.moe_select(z[:, :self.n_out], self.router_b, idx, wt, k, rule=self.rule, out_scale=self.route_scale)
@@ -164,25 +177,27 @@ class RoutedExperts(FeedForward):
         else:
             ops.moe_route(x, self.router, self.router_b, idx, wt, k)
         if not small:
-            ops.moe_sort(idx, self.n_out, group_off, pos_of_slot, row_of_pos)
+            ops.moe_sort(idx, self.n_out, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos)
         act = ws.rows("moe_act", T, k * self.ff, dt).view(n_slots, self.ff)
         y = ws.rows("moe_y", T, k * W, dt).view(n_slots, W)
         if self.library_ok and n_slots >= self.LIBRARY_FROM_SLOTS and normed_in is None:
             xs = ws.rows("moe_x_sorted", T, k * W, dt).view(n_slots, W)
             ops.gather_rows(x, row_of_pos, xs)
             ends = group_off[1:self.n + 1]        # (the places of identity units, behind the last expert's, are not computed)
-            ops.swiglu(F.grouped_mm(xs, self._w_gate_up_t, offs=ends), act)
+            ops.swiglu(F.grouped_mm(xs, self._w_gate_up_t, offs=ends), act, row_scale=wt_of_pos)
             y = F.grouped_mm(act, self._w_down_t, offs=ends)
         else:
             ops.gemm_grouped(x if normed_in is None else x.xw, self.w_gate_up, act, group_off=group_off, a_rows=row_of_pos, n_rows=n_slots,
-                             glu=True, row_scale=rstd)
+                             glu=True, row_scale=wt_of_pos if self.w_on_input else rstd, scale_by_place=self.w_on_input)
             ops.gemm_grouped(act, self.w_down, y, group_off=group_off, n_rows=n_slots)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         if tail is not None:
             return ops.moe_combine_resid(y, pos_of_slot, wt, shared, tail.resid, tail.scale, tail.norm.weight, tail.norm.eps,
                                          ws.rows("xw_ffn", T, W, dt), ws.rows("sumsq_ffn", T, (W + 15) // 16, torch.float32))
+        if routed:
+            return ops.RoutedRows(y, pos_of_slot, None if self.w_on_input else wt, k)
         out = ws.rows("moe_out", T, W, dt)
-        ops.moe_combine(y, pos_of_slot, wt, shared, out, group_off=group_off if self.n_id else None, n_real=self.n,
+        ops.moe_combine(y, pos_of_slot, None if self.w_on_input else wt, shared, out, top=k, group_off=group_off if self.n_id else None, n_real=self.n,
                         x=x if self.n_id else None, shared_gate=z[:, self.n_out] if self.has_sg else None)
         return out
 

@@ -10,6 +10,10 @@ afterwards, and the mask may be runs of `chunk` positions or a sliding `window`.
     o_h = softmax over j <= i (optionally with a sink of score 0 in the denominator) of the scores, times v
     y = W_o ([o_1 .. o_H] * sigmoid(g))                                           (the gate, one per column, is optional)
 
+Another way to weigh the keys (`weights` "sigmoid"): no softmax, o_h = sum over the visible j of sigmoid(score + pb_h) v, with
+pb one number per head (tensor `pb`). Another bias by distance (`distance_log`): the score loses r1_h ln(1 + r2_h (i - j))
+(tensors `r1`, `r2` [heads]); over a window it is unrolled at load into the same table by distance, pb joining it.
+
 Options: the values may be the keys as projected, before their norm (no v tensor); a mixer may read the keys and values that
 another run-order entry cached (no k, v tensors, no cache of its own); key size and value size may differ - heads are laid
 out at hd = max of the two rounded up to 16, the surplus columns zero, as `conv_attention` does.
@@ -18,7 +22,7 @@ The bias: table [rows, heads]; distances below rows/2 have a row each, the other
 scale that reaches the last row at distance `far`: bucket(n) = n for n < rows/2, else
 min(rows - 1, rows/2 + floor(ln(n / (rows/2)) / ln(far / (rows/2)) * (rows - rows/2))). At load it is unrolled into a float32
 table [far + 1, heads] by distance, constant from `far` on, which is what the attention kernels index.
-Tensors (under the part's prefix): q, k, v, g, o [out, in]; q.b, k.b, v.b; q.norm, k.norm [dim]; rel [rows, heads].
+Tensors (under the part's prefix): q, k, v, g, o [out, in]; q.b, k.b, v.b; q.norm, k.norm [dim]; rel [rows, heads]; r1, r2, pb [heads].
 """
 from __future__ import annotations
 
@@ -55,8 +59,10 @@ class QKNormAttention(Mixer):
     a value and with score 0 joins the softmax), output_gate, plain_kernel, prefill_kernel;
     norm_over ("head", the default, or "projection": q.norm has heads * qk_dim entries, k.norm kv_heads * qk_dim),
     position (PartSpec of a rotary encoding, with norm_over "projection"), chunk (runs of that many positions, counted from the
-    sequence's start; a query sees its own run) or window (a sliding window; its pages are given back behind it)."""
+    sequence's start; a query sees its own run) or window (a sliding window; its pages are given back behind it);
+    weights ("softmax", the default, or "sigmoid"), distance_log (with a window, instead of distance_bias)."""
     graph_safe = True
+    MAX_DISTANCES = 1 << 20                       # rows of an unrolled table by distance
 
     def __init__(self, params, prefix, dtype):
         super().__init__(params, prefix, dtype)
@@ -83,11 +89,21 @@ class QKNormAttention(Mixer):
         if qt and self.t_every < 1:
             raise ValueError("attention: the query temperature's step must be at least 1")
         self.sink_zero = bool(p.get("sink_zero", False))
+        kind = str(p.get("weights", "softmax"))
+        if kind not in ("softmax", "sigmoid"):
+            raise ValueError("attention: weights is 'softmax' or 'sigmoid'")
+        self.sigmoid, self.dist_log = kind == "sigmoid", bool(p.get("distance_log", False))
+        if self.sigmoid and self.sink_zero:
+            raise ValueError("attention: a sink belongs to a softmax")
+        if (self.sigmoid or self.dist_log) and (self.has_bias or p.get("window") is None):
+            raise ValueError("attention: sigmoid weights and a logarithmic bias by distance go with a window and without a learned table")
+        if (self.sigmoid or self.dist_log) and int(p["window"]) > self.MAX_DISTANCES:
+            raise ValueError(f"attention: a table by distance of {p['window']} rows (at most {self.MAX_DISTANCES})")
         self.norm_rows = str(p.get("norm_over", "head")) == "projection"
         if str(p.get("norm_over", "head")) not in ("head", "projection"):
             raise ValueError("attention: norm_over is 'head' or 'projection'")
         self.position = build_part("position", p.get("position") or PartSpec("none"), dtype)
-        if self.position.has_transform or (self.position.rot_dim and not self.norm_rows) or self.position.rot_dim > self.dk:
+        if self.position.interleaved or self.position.has_transform or (self.position.rot_dim and not self.norm_rows) or self.position.rot_dim > self.dk:
             raise ValueError("attention: a rotary table of at most qk_dim dimensions, with the norm over the projection")
         if self.norm_rows and (self.v_from_k or qt):
             raise ValueError("attention: the norm over the projection goes with values of their own and no query temperature")
@@ -108,7 +124,7 @@ class QKNormAttention(Mixer):
         self.proj = Linear(self.hidden, self.n_proj_pad, dtype)
         self.o_proj = Linear(self.nh * self.dv, self.hidden, dtype)
         self.core = PagedAttend(dtype, self.nh, self.nkv, self.hd, self.scale, self.window, bool(p.get("plain_kernel", False)),
-                                str(p.get("prefill_kernel", "auto")), chunk=self.chunk)
+                                str(p.get("prefill_kernel", "auto")), chunk=self.chunk, sigmoid=self.sigmoid)
         self.w_q = self.w_k = None
 
     def weight_specs(self) -> List[WeightSpec]:
@@ -127,6 +143,10 @@ class QKNormAttention(Mixer):
                     specs.append(WeightSpec("v.b", (self.nvv,), "vector", ("normal", 0.02)))
         if self.has_bias:
             specs.append(WeightSpec("rel", (-1 if self.bias_rows is None else self.bias_rows, self.nh), "vector", ("normal", 0.5), free=16))
+        if self.dist_log:
+            specs += [WeightSpec("r1", (self.nh,), "vector", ("ones_normal", 0.3)), WeightSpec("r2", (self.nh,), "vector", ("ones_normal", 0.3))]
+        if self.sigmoid:
+            specs.append(WeightSpec("pb", (self.nh,), "vector", ("normal", 1.0)))
         if self.gate:
             specs.append(WeightSpec("g", (self.nh * self.dv, H)))
         return specs
@@ -149,6 +169,14 @@ class QKNormAttention(Mixer):
         if self.has_bias:
             idx = torch.tensor(distance_buckets(int(t["rel"].shape[0]), self.bias_far), dtype=torch.long, device=dev)
             self.core.dist_bias = t["rel"].to(torch.float32)[idx].contiguous()          # [far + 1, heads]
+        if self.dist_log or self.sigmoid:         # by distance n inside the window: pb - r1 ln(1 + r2 n), each optional
+            n = torch.arange(int(self.window), dtype=torch.float64, device=dev)[:, None]
+            table = torch.zeros((int(self.window), self.nh), dtype=torch.float64, device=dev)
+            if self.dist_log:
+                table -= t["r1"].double()[None, :] * torch.log1p(t["r2"].double()[None, :] * n)
+            if self.sigmoid:
+                table += t["pb"].double()[None, :]
+            self.core.dist_bias = table.to(torch.float32).contiguous()
         if self.sink_zero:
             self.core.sink = torch.zeros(self.nh, dtype=torch.float32, device=dev)
         self.position.to_device(dev)

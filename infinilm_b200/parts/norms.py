@@ -52,5 +52,12 @@ class RMSNorm(Norm):
         new stream in the compute dtype."""
         ops.norm_add(resid, branch, self.weight, self.eps, scale, copy)
 
+    def norm_add_norm(self, resid, branch, next_norm, out):
+        """resid (f32 [T,H]) += norm(branch); then, with a `next_norm`, out = next_norm(resid). `branch`: rows or `ops.RoutedRows`."""
+        if next_norm is None:
+            ops.norm_add_norm(resid, branch, self.weight, self.eps)
+        else:
+            ops.norm_add_norm(resid, branch, self.weight, self.eps, next_norm.weight, next_norm.eps, out)
+
 
 register_part("norm", "rmsnorm", RMSNorm)

@@ -1,4 +1,4 @@
-"""Rotary position encodings: plain RoPE and LongRoPE, as frequency tables a mixer applies.
+"""Rotary position encodings: plain RoPE, LongRoPE and YaRN, as frequency tables a mixer applies.
 
 Parity with InfiniLM: `csrc/layers/rotary_embedding/rotary_embedding.cpp:50-113` (one rotary
 object from head_dim, rotary_dim, max positions, theta, scaling), `rope_scaling_creators.cpp:23-47`
@@ -11,6 +11,10 @@ max_position_embeddings exceeds original_max_position_embeddings, else `short_fa
 cos/sin are multiplied by sqrt(1 + ln(s) / ln(original_max)) with s = max/original (or `factor`
 when given and not 1) if s > 1. The choice depends on the configuration only, never on the
 length of the sequence at hand, so a position's encoding is the same however the work is cut.
+
+YaRN (Peng, Quesnelle, Fan, Shippole: "YaRN: Efficient Context Window Extension of Large Language Models") divides by `factor`
+the frequencies that turn fewer than `slow` times over the original length, keeps those that turn more than `fast` times,
+blends linearly between, and multiplies cosine and sine by 0.1 ln(factor) + 1.
 """
 from __future__ import annotations
 
@@ -41,19 +45,33 @@ def longrope_choice(short_factor, long_factor, original_max: int, max_pos: int, 
     return factors, mscale
 
 
+def yarn_inv_freq(rot_dim: int, theta: float, factor: float, original: float, fast: float, slow: float) -> List[float]:
+    def dim_of(turns: float) -> float:            # the (real-valued) index whose wavelength fits `original` that many times
+        return rot_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+    lo = max(math.floor(dim_of(fast)), 0)
+    hi = min(math.ceil(dim_of(slow)), rot_dim - 1)
+    out = []
+    for i, f in enumerate(rotary_inv_freq(rot_dim, theta, None)):
+        ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(f / factor * ramp + f * (1.0 - ramp))
+    return out
+
+
 class Rope(PositionEncoding):
-    """params: rot_dim, theta."""
+    """params: rot_dim, theta, interleaved (default False: dimension i pairs with i + rot_dim / 2)."""
 
     def __init__(self, params, prefix, dtype):
         super().__init__(params, prefix, dtype)
         self.rot_dim = int(params["rot_dim"])
         self.theta = float(params["theta"])
         self.mscale = 1.0
+        self.interleaved = bool(params.get("interleaved", False))
         self._table = rotary_inv_freq(self.rot_dim, self.theta, None)
         self.inv_freq = None
 
     def to_device(self, device):
-        self.inv_freq = torch.tensor(self._table, dtype=torch.float64).to(torch.float32).to(device)
+        self.freq64 = torch.tensor(self._table, dtype=torch.float64).to(device)
+        self.inv_freq = self.freq64.to(torch.float32)
 
 
 class LongRope(Rope):
@@ -73,6 +91,19 @@ class LongRope(Rope):
         self.inv_freq = None
 
 
+class YarnRope(Rope):
+    """params: rot_dim, theta, interleaved, factor, original (positions), fast, slow (turns over them)."""
+
+    def __init__(self, params, prefix, dtype):
+        super().__init__(params, prefix, dtype)
+        factor, original = float(params["factor"]), float(params["original"])
+        fast, slow = float(params["fast"]), float(params["slow"])
+        if min(factor, original, fast, slow) <= 0.0 or self.theta <= 0.0 or self.theta == 1.0:
+            raise ValueError("yarn: factor, original, fast, slow must be positive, theta positive and not 1")
+        self._table = yarn_inv_freq(self.rot_dim, self.theta, factor, original, fast, slow)
+        self.mscale = 0.1 * math.log(factor) + 1.0
+
+
 class NoPosition(PositionEncoding):
     """No position encoding (rot_dim 0)."""
 
@@ -83,4 +114,5 @@ class NoPosition(PositionEncoding):
 
 register_part("position", "rope", Rope)
 register_part("position", "longrope", LongRope)
+register_part("position", "yarn", YarnRope)
 register_part("position", "none", NoPosition)
