@@ -175,7 +175,7 @@ def timeline_step(args) -> int:
     raw = dict(CONFIG_05B if args.sizes == "0.5b" else CONFIG_8B)
     raw["num_hidden_layers"] = args.layers or 4
     if args.design != "default":                  # one of the pair of `--workload designs`, at the first of --design-sizes
-        pair = {"gopitar": gopitar_pair, "somipel": somipel_pair, "zokuzen": zokuzen_pair}.get(args.design, design_pair)
+        pair = {"gopitar": gopitar_pair, "somipel": somipel_pair, "zokuzen": zokuzen_pair, "zibinex": zibinex_pair}.get(args.design, design_pair)
         raw = pair(args.design_sizes.split(",")[0], args.layers or 4)[1 if args.design == "dense" else 0]
         raw["num_hidden_layers"] = args.layers or 4
     cfg = config_from_json(raw)
@@ -363,6 +363,29 @@ def zokuzen_pair(size: str, layers: int):
     return zk, nz
 
 
+def zibinex_pair(size: str, layers: int):
+    """(Zibinex configuration, Nirozen configuration of the same width, depth, heads, head size, cached latent width, vocabulary,
+    experts and ACTIVE feed-forward width: the framework's other design with latent attention over all keys and routed experts.)
+    Every other layer mixes by latent attention (of the cached width a quarter is the rotated key part), the others by sigmoid
+    attention over a window of 1,024 (2 kv heads); the first feed-forward is dense, the others route. (Nirozen's shared unit,
+    two experts wide, is two more chosen experts here: one at the small width.)"""
+    nz = design_pair(size, layers)[0]
+    W, V = nz["width"], nz["vocab"]
+    m0, f0 = nz["layers"][0]["mixer"], nz["layers"][0]["mlp"]
+    H, d, r, ff, sh = m0["heads"], m0["dim"], m0["kv_rank"], f0["expert"]["ff"], f0["shared"]["ff"]
+    top = f0["router"]["top"]
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": f0["router"]["experts"], "top": top + sh // ff}}
+    rd = r // 4
+    lat = {"heads": H, "dim": d, "rot_dim": rd, "vdim": d, "kv_rank": r - rd, "scale": (d + rd) ** -0.5,
+           "rot": {"dims": rd, "base": 1e4, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    att = {"heads": H, "kv_heads": 2, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": 1024}}
+    zb = {"architecture": "Zibinex", "vocab": V, "width": W, "norm": {"eps": 1e-5},
+          "layers": [{"type": "attention", "mixer": dict(att), "mlp": dict(moe)} if i % 2 else
+                     {"type": "latent_attention", "mixer": dict(lat), "mlp": dict(moe) if i else {"kind": "dense", "ff": top * ff + sh, "limit": 7.0}}
+                     for i in range(layers)]}
+    return zb, nz
+
+
 class OpTimer:
     """Brackets every kernel wrapper of `infinilm_b200.ops`, every library product of `Linear` and the library's grouped
     product with CUDA events on the launching stream, for steps that run eagerly; `table()` gives microseconds and calls per name."""
@@ -406,7 +429,7 @@ class OpTimer:
                      "gemm_tc5", "latent_norm_store", "moe_route", "moe_sort", "moe_combine", "gather_rows", "gemm_grouped", "short_conv",
                      "short_conv_state", "delta_prep", "matrix_state_scan", "group_norm_gate", "head_gate", "scaled_sum", "softcap", "silu_cols", "norm_add", "cast_rows",
                      "qk_norm_store", "gate_pack", "stabilized_gates", "hyper_step", "qk_rows_norm_rope_store", "token_shift_mix",
-                     "double_exp_decay", "tanh_rows", "moe_select", "moe_route_sort_small"):
+                     "double_exp_decay", "tanh_rows", "moe_select", "moe_route_sort_small", "norm_add_norm", "latent_rope_store"):
             self._wrap(ops, name)
         self._wrap(Linear, "__call__", "linear")
         if hasattr(F, "grouped_mm"):
@@ -445,8 +468,8 @@ def run_designs(args) -> int:
         rec = {"workload": "designs", "size": size, "layers": L, "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src}}
         family = getattr(args, "design_family", "nirozen")
         rec["design"] = family
-        pair = {"gopitar": gopitar_pair, "somipel": somipel_pair, "zokuzen": zokuzen_pair}.get(family, design_pair)
-        for which, raw in zip((family, {"somipel": "gopitar", "zokuzen": "nirozen"}.get(family, "dense_gqa")), pair(size, L)):
+        pair = {"gopitar": gopitar_pair, "somipel": somipel_pair, "zokuzen": zokuzen_pair, "zibinex": zibinex_pair}.get(family, design_pair)
+        for which, raw in zip((family, {"somipel": "gopitar", "zokuzen": "nirozen", "zibinex": "nirozen"}.get(family, "dense_gqa")), pair(size, L)):
             cfg = config_from_json(raw)
             B = 64
             eng = Engine.from_tensors(cfg, random_tensors(cfg, 0, "cuda:0"), dtype="bfloat16", page_size=PAGE,
@@ -547,11 +570,11 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 and 64 points")
     ap.add_argument("--no-graph", action="store_true", help="do not replay decode steps as CUDA graphs")
     ap.add_argument("--points", type=str, default="1,64", help="batch sizes of the extra decode points")
-    ap.add_argument("--design", choices=["default", "nirozen", "gopitar", "somipel", "zokuzen", "dense"], default="default",
+    ap.add_argument("--design", choices=["default", "nirozen", "gopitar", "somipel", "zokuzen", "zibinex", "dense"], default="default",
                     help="--timeline: the step of one of the pair of --workload designs instead of the benchmark model")
-    ap.add_argument("--design-family", choices=["nirozen", "gopitar", "somipel", "zokuzen"], default="nirozen",
+    ap.add_argument("--design-family", choices=["nirozen", "gopitar", "somipel", "zokuzen", "zibinex"], default="nirozen",
                     help="--workload designs: which design stands beside the dense GQA model of equal size (somipel: beside gopitar; "
-                         "zokuzen: beside nirozen)")
+                         "zokuzen, zibinex: beside nirozen)")
     ap.add_argument("--design-sizes", type=str, default="1k,2k", help="--workload designs: layer sizes to run (1k, 2k, 4k)")
     ap.add_argument("--workload", choices=["default", "long_context", "continuous", "designs"], default="default",
                     help="default: the benchmark line. long_context: 8 requests x 16,384-token prompts at 8B sizes, prompt "

@@ -9,17 +9,17 @@
 // positions max(0, p - window + 1) .. p (window <= 0: all). Query head j reads kv head j / (nh / nkv).
 // With `dist_bias` (f32 [dist_far + 1][heads]) the scaled score of a key n positions back gets dist_bias[min(n, dist_far)][head]
 // added: a learned bias by distance that is constant from dist_far on.
-// `sigmoid`: no softmax - a visible key's weight is the sigmoid of its (scaled, biased) score, and the weights are not
+// SIG: no softmax - a visible key's weight is the sigmoid of its (scaled, biased) score, and the weights are not
 // normalised over the keys.
 #include "common.cuh"
 
 // A lane holds head_dim / 32 elements of the query and of the output: 8 (head_dim <= 256) or 32 (<= 1024).
-template <typename TA, int AP_MAX_PER_LANE>
+template <typename TA, int AP_MAX_PER_LANE, bool SIG>
 __global__ void attn_plain_kernel(const TA* __restrict__ qkv, int row_stride, TA* __restrict__ out,
                                   const TA* __restrict__ cache, const int* __restrict__ block_table, int bt_stride,
                                   const int* __restrict__ tok_pos, const int* __restrict__ tok_entry, int page_size,
                                   int nh, int nkv, int hd, float scale, int window, const float* __restrict__ sink,
-                                  const float* __restrict__ dist_bias, int dist_far, int sigmoid) {
+                                  const float* __restrict__ dist_bias, int dist_far) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int j = blockIdx.y * (blockDim.x >> 5) + warp;
     const int t = blockIdx.x;
@@ -51,9 +51,18 @@ __global__ void attn_plain_kernel(const TA* __restrict__ qkv, int row_stride, TA
         }
         dot = il_warp_sum(dot) * scale;
         if (dist_bias) dot += dist_bias[(size_t)min(pos - kp, dist_far) * nh + j];
-        const float mn = sigmoid ? 0.f : fmaxf(m, dot);
-        const float corr = sigmoid ? 1.f : expf(m - mn);  // exp(-inf) = 0 on the first key
-        const float p = sigmoid ? 1.f / (1.f + expf(-dot)) : expf(dot - mn);
+        if constexpr (SIG) {
+            const float w = 1.f / (1.f + expf(-dot));
+#pragma unroll
+            for (int r = 0; r < AP_MAX_PER_LANE; ++r) {
+                const int d = lane + 32 * r;
+                if (d < hd) acc[r] = fmaf(w, il_to_f(vrow[d]), acc[r]);
+            }
+            continue;
+        }
+        const float mn = fmaxf(m, dot);
+        const float corr = expf(m - mn);  // exp(-inf) = 0 on the first key
+        const float p = expf(dot - mn);
         l = l * corr + p;
 #pragma unroll
         for (int r = 0; r < AP_MAX_PER_LANE; ++r) {
@@ -64,7 +73,7 @@ __global__ void attn_plain_kernel(const TA* __restrict__ qkv, int row_stride, TA
     }
     TA* orow = out + (size_t)t * nh * hd + (size_t)j * hd;
     if (sink) l += expf(sink[j] - m);             // (+inf when the sink towers over every score: the row is then zero)
-    const float inv = sigmoid ? 1.f : 1.f / l;
+    const float inv = SIG ? 1.f : 1.f / l;
 #pragma unroll
     for (int r = 0; r < AP_MAX_PER_LANE; ++r) {
         const int d = lane + 32 * r;
@@ -82,9 +91,13 @@ IL_EXPORT int il_attn_plain(const void* qkv, int act_kind, int row_stride, void*
     if (hd > 1024) return IL_UNSUPPORTED;
     const int warps = 4;
     dim3 grid(T, (nh + warps - 1) / warps);
-#define AP_LAUNCH(TA, N)                                                                                                                \
-    attn_plain_kernel<TA, N><<<grid, warps * 32, 0, stream>>>((const TA*)qkv, row_stride, (TA*)out, (const TA*)cache, block_table, bt_stride, \
-                                                              tok_pos, tok_entry, page_size, nh, nkv, hd, scale, window, sink, dist_bias, dist_far, sigmoid)
+#define AP_LAUNCH1(TA, N, S)                                                                                                                \
+    attn_plain_kernel<TA, N, S><<<grid, warps * 32, 0, stream>>>((const TA*)qkv, row_stride, (TA*)out, (const TA*)cache, block_table, bt_stride, \
+                                                              tok_pos, tok_entry, page_size, nh, nkv, hd, scale, window, sink, dist_bias, dist_far)
+#define AP_LAUNCH(TA, N)                                            \
+    do {                                                            \
+        if (sigmoid) AP_LAUNCH1(TA, N, true); else AP_LAUNCH1(TA, N, false); \
+    } while (0)
     if (act_kind == IL_F32) {
         if (hd <= 256) AP_LAUNCH(float, 8); else AP_LAUNCH(float, 32);
     } else if (act_kind == IL_BF16) {
@@ -92,6 +105,7 @@ IL_EXPORT int il_attn_plain(const void* qkv, int act_kind, int row_stride, void*
     } else
         return IL_BAD_ARG;
 #undef AP_LAUNCH
+#undef AP_LAUNCH1
     IL_LAUNCH_CHECK();
     return IL_OK;
 }

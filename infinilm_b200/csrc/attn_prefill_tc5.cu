@@ -32,6 +32,8 @@
 //   SIG: no softmax - a visible key's weight is the sigmoid of its (scaled, biased) score, not normalised over the keys. No
 //   maximum, no rescaling of O, no row sums; a score costs an exponential and half a reciprocal (two scores share one:
 //   1/a = b/(ab)), so the special-function unit is the busier half of a tile.
+//   LOGB (with SIG): the bias by distance is pb_h - r1_h ln(1 + r2_h n), made here of three numbers per head instead of read
+//   from a table: a logarithm more per score, no loads (64 a row and tile) and no registers for them.
 //
 //   Pages past the entry's last page are read as the last page again (finite values the mask removes).
 //   Every mbarrier wait is bounded; one that runs out sets *status and all roles leave their loops.
@@ -82,17 +84,23 @@ __device__ __forceinline__ float pt_ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
     return y;
 }
+__device__ __forceinline__ float pt_lg2(float x) {
+    float y;
+    asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ uint32_t pt_pack(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <bool SIG>
+template <bool SIG, bool LOGB>
 __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5_kernel(
     const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* __restrict__ qkv, int row_stride,
     __nv_bfloat16* __restrict__ out, const int* __restrict__ block_table, int bt_stride, const int* __restrict__ entry_qstart,
     const int* __restrict__ entry_kvlen, int first_entry, int n_entries, int nh, int nkv, float scale_log2, int window, int tpt,
-    int* __restrict__ status, const float* __restrict__ sink, const float* __restrict__ dist_bias, int dist_far, float inv_scale) {
+    int* __restrict__ status, const float* __restrict__ sink, const float* __restrict__ dist_bias, int dist_far, float inv_scale,
+    const float* __restrict__ log_bias) {
     extern __shared__ __align__(1024) unsigned char smem[];
     if (t5_smem(smem) & 1023u) {                  // the swizzled tiles need 1 KB alignment; dynamic shared memory starts on it
         if (threadIdx.x == 0) atomicExch(status, 30);
@@ -282,6 +290,8 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
         // a bias by distance: this row's column of the table (bias[min(n, dist_far)][head]: a warp's rows are the heads of a few
         // neighbouring tokens, so what it reads for one key lies together) and its value from dist_far on,
         // both as they join the unscaled score (bias / scale)
+        const float lb_r1 = LOGB ? log_bias[g * G + hh] : 0.f, lb_r2 = LOGB ? log_bias[nh + g * G + hh] : 0.f;
+        const float lb_pb = LOGB ? log_bias[2 * nh + g * G + hh] * 1.4426950408889634f : 0.f;
         const float* db_row = dist_bias ? dist_bias + g * G + hh : nullptr;
         const float db_far = dist_bias ? db_row[(size_t)dist_far * nh] * inv_scale : 0.f;
         for (int j = 0; j < n_tiles; ++j) {
@@ -297,7 +307,7 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
             __syncwarp();
             if (lane == 0) t5_mbar_arrive(s_free0 + 8 * b);
             const int kb = (page_first + j * PT_TILE_PAGES) * PT_PAGE;
-            if (dist_bias) {
+            if (!LOGB && dist_bias) {
                 if (rpos - (kb + PT_KEYS - 1) >= dist_far) {  // the whole tile lies beyond dist_far for this row: a constant
 #pragma unroll
                     for (int c = 0; c < PT_KEYS; ++c) sv[c] = __float_as_uint(__uint_as_float(sv[c]) + db_far);
@@ -323,10 +333,15 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
             if constexpr (SIG) {
                 // 1 / (1 + 2^-v): the exponent is kept below 60 so that the product of two denominators stays finite, and a key
                 // that the mask took out (-inf) is set to zero
+                // (in base 2: the sigmoid's exponent is -(s scale + bias) log2 e, and ln(x) log2 e = log2 x; beyond the row's own position
+                // the logarithm's argument may be anything - such a key is masked)
+                const float y0 = LOGB ? fmaf(lb_r2, (float)(rpos - kb), 1.f) : 0.f;
 #pragma unroll
                 for (int c = 0; c < PT_KEYS; c += 2) {
                     const float s0 = __uint_as_float(sv[c]), s1 = __uint_as_float(sv[c + 1]);
-                    const float a = 1.f + pt_ex2(fminf(s0 * -scale_log2, 60.f)), bb = 1.f + pt_ex2(fminf(s1 * -scale_log2, 60.f));
+                    const float e0 = LOGB ? fmaf(s0, -scale_log2, fmaf(lb_r1, pt_lg2(fmaf((float)-c, lb_r2, y0)), -lb_pb)) : s0 * -scale_log2;
+                    const float e1 = LOGB ? fmaf(s1, -scale_log2, fmaf(lb_r1, pt_lg2(fmaf((float)(-c - 1), lb_r2, y0)), -lb_pb)) : s1 * -scale_log2;
+                    const float a = 1.f + pt_ex2(fminf(e0, 60.f)), bb = 1.f + pt_ex2(fminf(e1, 60.f));
                     const float rr = __fdividef(1.f, a * bb);
                     sv[c >> 1] = pt_pack(s0 == -INFINITY ? 0.f : rr * bb, s1 == -INFINITY ? 0.f : rr * a);
                 }
@@ -437,9 +452,11 @@ IL_EXPORT int il_attn_prefill_tc5_rows() { return PT_ROWS; }
 IL_EXPORT int il_attn_prefill_tc5(const void* qkv, int row_stride, void* out, const void* kv_map, const int* block_table,
                                   int bt_stride, const int* entry_qstart, const int* entry_kvlen, int page_size, int first_entry,
                                   int n_entries, int n_tiles_total, int nh, int nkv, int hd, float scale, int window, int* status,
-                                  const float* sink, const float* dist_bias, int dist_far, int sigmoid, cudaStream_t stream) {
+                                  const float* sink, const float* dist_bias, int dist_far, int sigmoid, const float* log_bias,
+                                  cudaStream_t stream) {
     if (n_tiles_total <= 0 || first_entry >= n_entries) return IL_OK;
     if (dist_bias && (dist_far < 0 || (long long)(dist_far + 1) * nh > 0x7fffffffLL)) return IL_BAD_ARG;
+    if (log_bias && (!sigmoid || dist_bias)) return IL_BAD_ARG;
     if (sigmoid && sink) return IL_BAD_ARG;       // a sink is a term of a softmax's denominator
     if (hd != HEAD_DIM || page_size != PT_PAGE || !kv_map || !status) return IL_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) return IL_BAD_ARG;
@@ -451,7 +468,7 @@ IL_EXPORT int il_attn_prefill_tc5(const void* qkv, int row_stride, void* out, co
     static bool attr_set[64];
     if (dev >= 0 && dev < 64 && !attr_set[dev]) {
         cudaError_t e = cudaSuccess;
-        for (auto k : {attn_prefill_tc5_kernel<false>, attn_prefill_tc5_kernel<true>}) {
+        for (auto k : {attn_prefill_tc5_kernel<false, false>, attn_prefill_tc5_kernel<true, false>, attn_prefill_tc5_kernel<true, true>}) {
             if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, PT_SMEM);
             if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
         }
@@ -461,9 +478,9 @@ IL_EXPORT int il_attn_prefill_tc5(const void* qkv, int row_stride, void* out, co
     CUtensorMap map;
     memcpy(&map, kv_map, sizeof(map));
     dim3 grid(n_tiles_total, nkv);
-    (sigmoid ? attn_prefill_tc5_kernel<true> : attn_prefill_tc5_kernel<false>)<<<grid, PT_THREADS, PT_SMEM, stream>>>(
+    (log_bias ? attn_prefill_tc5_kernel<true, true> : sigmoid ? attn_prefill_tc5_kernel<true, false> : attn_prefill_tc5_kernel<false, false>)<<<grid, PT_THREADS, PT_SMEM, stream>>>(
         map, (const __nv_bfloat16*)qkv, row_stride, (__nv_bfloat16*)out, block_table, bt_stride, entry_qstart, entry_kvlen,
-        first_entry, n_entries, nh, nkv, scale * 1.4426950408889634f, window, PT_ROWS / G, status, sink, dist_bias, dist_far, 1.f / scale);
+        first_entry, n_entries, nh, nkv, scale * 1.4426950408889634f, window, PT_ROWS / G, status, sink, dist_bias, dist_far, 1.f / scale, log_bias);
     IL_LAUNCH_CHECK();
     return IL_OK;
 }

@@ -81,7 +81,11 @@ IL_EXPORT int il_latent_norm_store(const void* proj, int act_kind, int row_strid
 // Angles are made in double precision and reduced to one turn before sine and cosine are taken in f32: an f32 product of
 // position and frequency would be off by a rounding of the whole angle. Norm and rotation f32. One block per token.
 #define LR_MAX_ROT 1024
-template <typename TA>
+__device__ __forceinline__ float2 lr_ld2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 lr_ld2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ void lr_st2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+__device__ __forceinline__ void lr_st2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
+template <typename TA, bool VEC>
 __global__ void latent_rope_store_kernel(const TA* proj, int row_stride, int off_q, int nh, int qd, int off_b, int n_b, int rd, int hd,
                                          const void* __restrict__ w_b, int w_kind, float eps, int rot, const double* __restrict__ freq, float mscale,
                                          int interleaved, TA* __restrict__ q_out, const int* __restrict__ tok_pos, const int* __restrict__ tok_entry,
@@ -98,9 +102,8 @@ __global__ void latent_rope_store_kernel(const TA* proj, int row_stride, int off
     }
     const int half = rot >> 1;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
-        const double turn = 6.283185307179586476925;
         double a = (double)pos * freq[i];
-        a -= turn * rint(a / turn);
+        a -= 6.283185307179586476925 * rint(a * 0.15915494309189533577);
         float s, c;
         sincosf((float)a, &s, &c);
         s_sin[i] = s * mscale, s_cos[i] = c * mscale;
@@ -121,6 +124,34 @@ __global__ void latent_rope_store_kernel(const TA* proj, int row_stride, int off
         const float a = il_to_f(x[d]), b = il_to_f(x[mate]), s = s_sin[i], c = s_cos[i];
         return low ? a * c - b * s : a * c + b * s;
     };
+    const int tail = hd - n_b;
+    if (VEC) {                                    // two neighbouring columns a thread: with interleaved pairs, a pair
+        auto turned2 = [&](const TA* x, int d) -> float2 {
+            if (d >= rd) return make_float2(0.f, 0.f);
+            const float2 v = lr_ld2(x + d);
+            if (d >= rot) return v;
+            const float s = s_sin[d >> 1], c = s_cos[d >> 1];
+            return make_float2(v.x * c - v.y * s, v.y * c + v.x * s);
+        };
+        if (kdst)
+            for (int i = 2 * threadIdx.x; i < hd; i += 2 * blockDim.x) {
+                float2 f;
+                if (i < n_b) {
+                    f = lr_ld2(row + off_b + i);
+                    f.x *= rb * il_load_any(w_b, w_kind, i), f.y *= rb * il_load_any(w_b, w_kind, i + 1);
+                } else {
+                    f = turned2(row + off_b + n_b, i - n_b);
+                }
+                lr_st2(kdst + i, f);
+                lr_st2(kdst + plane + i, f);
+            }
+        const int t2 = tail >> 1;
+        for (int idx = threadIdx.x; idx < nh * t2; idx += blockDim.x) {
+            const int j = idx / t2, d = 2 * (idx - j * t2);
+            lr_st2(q_out + ((size_t)t * nh + j) * hd + n_b + d, turned2(row + off_q + (size_t)j * (qd + rd) + qd, d));
+        }
+        return;
+    }
     if (kdst) {
         for (int i = threadIdx.x; i < hd; i += blockDim.x) {
             const float f = i < n_b ? il_to_f(row[off_b + i]) * rb * il_load_any(w_b, w_kind, i) : i < n_b + rd ? turned(row + off_b + n_b, i - n_b) : 0.f;
@@ -129,7 +160,6 @@ __global__ void latent_rope_store_kernel(const TA* proj, int row_stride, int off
             kdst[plane + i] = v;
         }
     }
-    const int tail = hd - n_b;
     for (int idx = threadIdx.x; idx < nh * tail; idx += blockDim.x) {
         const int j = idx / tail, d = idx - j * tail;
         q_out[((size_t)t * nh + j) * hd + n_b + d] = il_from_f<TA>(d < rd ? turned(row + off_q + (size_t)j * (qd + rd) + qd, d) : 0.f);
@@ -146,15 +176,19 @@ IL_EXPORT int il_latent_rope_store(const void* proj, int act_kind, int row_strid
     if (rot > LR_MAX_ROT) return IL_UNSUPPORTED;
     const int work = hd + nh * (hd - n_b);
     const int threads = work >= 1024 ? 256 : 128;
-    if (act_kind == IL_F32)
-        IL_LAUNCH(latent_rope_store_kernel<float>, T, threads, 0, stream, (const float*)proj, row_stride, off_q, nh, qd, off_b, n_b, rd, hd, w_b, w_kind,
-                  eps, rot, freq, mscale, interleaved, (float*)q_out, tok_pos, tok_entry, block_table, bt_stride, (float*)cache, page_size);
-    else if (act_kind == IL_BF16)
-        IL_LAUNCH(latent_rope_store_kernel<__nv_bfloat16>, T, threads, 0, stream, (const __nv_bfloat16*)proj, row_stride, off_q, nh, qd, off_b, n_b, rd,
-                  hd, w_b, w_kind, eps, rot, freq, mscale, interleaved, (__nv_bfloat16*)q_out, tok_pos, tok_entry, block_table, bt_stride,
-                  (__nv_bfloat16*)cache, page_size);
-    else
+    // two columns a thread: every segment starts on an even column of rows of even length, pairs are neighbours (or nothing turns)
+    const bool vec = ((row_stride | off_q | qd | rd | off_b | n_b | hd) & 1) == 0 && (interleaved || rot == 0) &&
+                     (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache) & 7) == 0;
+#define LR_GO(TA, VEC)                                                                                                                      \
+    IL_LAUNCH((latent_rope_store_kernel<TA, VEC>), T, threads, 0, stream, (const TA*)proj, row_stride, off_q, nh, qd, off_b, n_b, rd, hd, w_b, \
+              w_kind, eps, rot, freq, mscale, interleaved, (TA*)q_out, tok_pos, tok_entry, block_table, bt_stride, (TA*)cache, page_size)
+    if (act_kind == IL_F32) {
+        if (vec) LR_GO(float, true); else LR_GO(float, false);
+    } else if (act_kind == IL_BF16) {
+        if (vec) LR_GO(__nv_bfloat16, true); else LR_GO(__nv_bfloat16, false);
+    } else
         return IL_BAD_ARG;
+#undef LR_GO
     IL_LAUNCH_CHECK();
     return IL_OK;
 }

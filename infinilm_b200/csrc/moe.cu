@@ -246,16 +246,26 @@ __global__ void __launch_bounds__(WARPS * 32) moe_select_kernel(const float* __r
 
 // The body of the sort, by one whole block; `sh`: 2 * E ints of shared memory. (idx is not declared __restrict__: the
 // fused kernel below reads what its own warps have just written.) `wt_of_pos` (or null) receives every place's weight: where a
-// choice's weight belongs to the expert's input, the products take it as a factor per place.
+// choice's weight belongs to the expert's input, the products take it as a factor per place. row_of_pos null: a kernel behind this
+// one fills in what lies in the order of the places.
 __device__ __forceinline__ void moe_sort_body(int* sh, const int* idx, int n_slots, int top, int E, int* __restrict__ group_off,
                                               int* __restrict__ pos_of_slot, int* __restrict__ row_of_pos, const float* wt, float* __restrict__ wt_of_pos) {
     int* cnt = sh;
     int* cur = sh + E;
     for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
     __syncthreads();
-    for (int i = threadIdx.x; i < n_slots; i += blockDim.x) {
-        const int e = idx[i];
-        if (e >= 0 && e < E) atomicAdd(&cnt[e], 1);
+    // (SL slots of a thread asked for at a time: one after the other they are a chain of round trips to memory)
+    constexpr int SL = 8;
+    for (int i0 = threadIdx.x; i0 < n_slots; i0 += SL * blockDim.x) {
+        int e[SL];
+#pragma unroll
+        for (int u = 0; u < SL; ++u) {
+            const int i = i0 + u * blockDim.x;
+            e[u] = i < n_slots ? idx[i] : -1;
+        }
+#pragma unroll
+        for (int u = 0; u < SL; ++u)
+            if (e[u] >= 0 && e[u] < E) atomicAdd(&cnt[e[u]], 1);
     }
     __syncthreads();
     if (threadIdx.x == 0) {
@@ -269,15 +279,41 @@ __device__ __forceinline__ void moe_sort_body(int* sh, const int* idx, int n_slo
     }
     __syncthreads();
     // the order of the rows inside an expert's range is whatever the atomics give: a row's result does not depend on it
-    for (int i = threadIdx.x; i < n_slots; i += blockDim.x) {
-        const int e = idx[i];
-        if (e >= 0 && e < E) {
-            const int p = atomicAdd(&cur[e], 1);
-            pos_of_slot[i] = p;
-            row_of_pos[p] = i / top;
-            if (wt_of_pos) wt_of_pos[p] = wt[i];
+    for (int i0 = threadIdx.x; i0 < n_slots; i0 += SL * blockDim.x) {
+        int e[SL];
+        float w[SL];
+#pragma unroll
+        for (int u = 0; u < SL; ++u) {
+            const int i = i0 + u * blockDim.x;
+            e[u] = i < n_slots ? idx[i] : -1;
+            w[u] = (wt_of_pos && i < n_slots) ? wt[i] : 0.f;
+        }
+#pragma unroll
+        for (int u = 0; u < SL; ++u) {
+            const int i = i0 + u * blockDim.x;
+            if (e[u] >= 0 && e[u] < E) {
+                const int p = atomicAdd(&cur[e[u]], 1);
+                pos_of_slot[i] = p;
+                if (row_of_pos) row_of_pos[p] = i / top;
+                if (wt_of_pos) wt_of_pos[p] = w[u];
+            } else if (i < n_slots) {
+                pos_of_slot[i] = -1;              // (no expert: nothing stands anywhere for it)
+            }
         }
     }
+}
+
+// The scattered half of a large sort by as many SMs as there are (one SM takes a clock and more per stored word: 20 us at 16,384
+// slots): every place learns its slot's token and weight.
+__global__ void moe_places_kernel(const int* pos_of_slot, int n_slots, int top, int* __restrict__ row_of_pos, const float* wt,
+                                  float* __restrict__ wt_of_pos) {
+    il_pdl_begin();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n_slots) return;
+    const int p = pos_of_slot[i];
+    if (p < 0) return;
+    row_of_pos[p] = i / top;
+    if (wt_of_pos) wt_of_pos[p] = wt[i];
 }
 
 __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* idx, int n_slots, int top, int E, int* __restrict__ group_off,
@@ -593,7 +629,12 @@ IL_EXPORT int il_moe_sort(const int* idx, int n_slots, int top, int E, int* grou
     if (E <= 0 || top <= 0 || n_slots < 0 || (wt_of_pos && !wt)) return IL_BAD_ARG;
     const size_t smem = (size_t)2 * E * sizeof(int);
     if (smem > 48 * 1024) return IL_UNSUPPORTED;
-    IL_LAUNCH(moe_sort_kernel, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
+    if (n_slots >= 4096) {
+        IL_LAUNCH(moe_sort_kernel, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, (int*)nullptr, (const float*)nullptr, (float*)nullptr);
+        IL_LAUNCH(moe_places_kernel, (n_slots + 255) / 256, 256, 0, stream, (const int*)pos_of_slot, n_slots, top, row_of_pos, wt, wt_of_pos);
+    } else {
+        IL_LAUNCH(moe_sort_kernel, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
+    }
     IL_LAUNCH_CHECK();
     return IL_OK;
 }

@@ -4,7 +4,7 @@
 //   k_g <- k_g / sqrt(mean(k_g^2) + eps) * w_k                     -> the token's slot of the cache, K plane
 //   v_g                                                            -> the V plane: the value columns, or the key columns as
 //                                                                     projected, before the norm (a mixer whose values are its keys)
-// all in f32; w_q and w_k are one vector each, shared by the heads. Heads are laid out at hd >= key size, value size: the
+// all in f32 - with `bias` (f32, one per column of the projection, or null) added to q, k and v first; w_q and w_k are one vector each, shared by the heads. Heads are laid out at hd >= key size, value size: the
 // surplus columns are written as zeros (a zero column adds nothing to a score). A mixer that reads another layer's cache
 // gives no key columns (k_off < 0): only its queries are normed.
 // Cache layout of one layer: [page][0=K,1=V][kv head][slot in page][hd]. One warp per (token, head).
@@ -25,6 +25,10 @@ __device__ __forceinline__ void qn_st4(__nv_bfloat16* p, float4 v) {
     u.y = *reinterpret_cast<const uint32_t*>(&b);
     *reinterpret_cast<uint2*>(p) = u;
 }
+__device__ __forceinline__ float4 qn_b4(float4 a, const float* b, int d) {      // a + the biases of its four columns
+    a.x += b[d], a.y += b[d + 1], a.z += b[d + 2], a.w += b[d + 3];
+    return a;
+}
 __device__ __forceinline__ float4 qn_w4(const void* w, int kind, int d) {
     return make_float4(il_load_any(w, kind, d), il_load_any(w, kind, d + 1), il_load_any(w, kind, d + 2), il_load_any(w, kind, d + 3));
 }
@@ -32,12 +36,13 @@ __device__ __forceinline__ float4 qn_w4(const void* w, int kind, int d) {
 // The form for sizes and offsets that are multiples of 4 (rows, segments and heads then start on 8- or 16-byte borders): the
 // lanes hold 4 neighbouring columns instead of every 32nd (the sum of squares is gathered in another order). VEC 1 is the form for
 // every size.
-template <typename TA, int VEC>
+template <typename TA, int VEC, bool BIAS>
 __global__ void qk_norm_store_kernel(const TA* proj, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int dk, int dv, int hd,
                                      const void* __restrict__ wq, const void* __restrict__ wk, int w_kind, float eps, float t_coef,
                                      int t_every, TA* __restrict__ q_out, const int* __restrict__ tok_pos,
                                      const int* __restrict__ tok_entry, const int* __restrict__ block_table, int bt_stride,
-                                     TA* __restrict__ cache, int page_size, int T) {
+                                     TA* __restrict__ cache, int page_size, int T,
+                                     const float* __restrict__ bias) {
     const int jobs = nh + (k_off >= 0 ? 2 * nkv : 0);
     const long long wid = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
     const int lane = threadIdx.x & 31;
@@ -48,16 +53,19 @@ __global__ void qk_norm_store_kernel(const TA* proj, int ld, int q_off, int k_of
     const TA* row = proj + (size_t)t * ld;
     if (j < nh) {                                 // a query head
         const TA* x = row + q_off + (size_t)j * dk;
+        const float* bx = BIAS ? bias + q_off + (size_t)j * dk : nullptr;
         TA* o = q_out + ((size_t)t * nh + j) * hd;
         float ss = 0.f;
         if (VEC == 4) {
             for (int d = 4 * lane; d < dk; d += 128) {
-                const float4 a = qn_ld4(x + d);
+                float4 a = qn_ld4(x + d);
+                if (BIAS) a = qn_b4(a, bx, d);
                 ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
             }
         } else {
             for (int d = lane; d < dk; d += 32) {
-                const float a = il_to_f(x[d]);
+                float a = il_to_f(x[d]);
+                if (BIAS) a += bx[d];
                 ss += a * a;
             }
         }
@@ -70,12 +78,13 @@ __global__ void qk_norm_store_kernel(const TA* proj, int ld, int q_off, int k_of
                 if (d < dk) {
                     const float4 w = qn_w4(wq, w_kind, d);
                     a = qn_ld4(x + d);
+                    if (BIAS) a = qn_b4(a, bx, d);
                     a.x *= r * w.x, a.y *= r * w.y, a.z *= r * w.z, a.w *= r * w.w;
                 }
                 qn_st4(o + d, a);
             }
         } else {
-            for (int d = lane; d < hd; d += 32) o[d] = il_from_f<TA>(d < dk ? il_to_f(x[d]) * r * il_load_any(wq, w_kind, d) : 0.f);
+            for (int d = lane; d < hd; d += 32) o[d] = il_from_f<TA>(d < dk ? (BIAS ? il_to_f(x[d]) + bx[d] : il_to_f(x[d])) * r * il_load_any(wq, w_kind, d) : 0.f);
         }
         return;
     }
@@ -87,15 +96,18 @@ __global__ void qk_norm_store_kernel(const TA* proj, int ld, int q_off, int k_of
     TA* dst = cache + (((size_t)page * 2 + (is_k ? 0 : 1)) * nkv + g) * (size_t)page_size * hd + (size_t)(pos % page_size) * hd;
     if (is_k) {
         const TA* x = row + k_off + (size_t)g * dk;
+        const float* bx = BIAS ? bias + k_off + (size_t)g * dk : nullptr;
         float ss = 0.f;
         if (VEC == 4) {
             for (int d = 4 * lane; d < dk; d += 128) {
-                const float4 a = qn_ld4(x + d);
+                float4 a = qn_ld4(x + d);
+                if (BIAS) a = qn_b4(a, bx, d);
                 ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
             }
         } else {
             for (int d = lane; d < dk; d += 32) {
-                const float a = il_to_f(x[d]);
+                float a = il_to_f(x[d]);
+                if (BIAS) a += bx[d];
                 ss += a * a;
             }
         }
@@ -107,19 +119,21 @@ __global__ void qk_norm_store_kernel(const TA* proj, int ld, int q_off, int k_of
                 if (d < dk) {
                     const float4 w = qn_w4(wk, w_kind, d);
                     a = qn_ld4(x + d);
+                    if (BIAS) a = qn_b4(a, bx, d);
                     a.x *= r * w.x, a.y *= r * w.y, a.z *= r * w.z, a.w *= r * w.w;
                 }
                 qn_st4(dst + d, a);
             }
         } else {
-            for (int d = lane; d < hd; d += 32) dst[d] = il_from_f<TA>(d < dk ? il_to_f(x[d]) * r * il_load_any(wk, w_kind, d) : 0.f);
+            for (int d = lane; d < hd; d += 32) dst[d] = il_from_f<TA>(d < dk ? (BIAS ? il_to_f(x[d]) + bx[d] : il_to_f(x[d])) * r * il_load_any(wk, w_kind, d) : 0.f);
         }
     } else {
         const TA* x = row + v_off + (size_t)g * dv;
+        const float* bx = BIAS ? bias + v_off + (size_t)g * dv : nullptr;
         if (VEC == 4) {
-            for (int d = 4 * lane; d < hd; d += 128) qn_st4(dst + d, d < dv ? qn_ld4(x + d) : make_float4(0.f, 0.f, 0.f, 0.f));
+            for (int d = 4 * lane; d < hd; d += 128) qn_st4(dst + d, d < dv ? (BIAS ? qn_b4(qn_ld4(x + d), bx, d) : qn_ld4(x + d)) : make_float4(0.f, 0.f, 0.f, 0.f));
         } else {
-            for (int d = lane; d < hd; d += 32) dst[d] = d < dv ? x[d] : il_from_f<TA>(0.f);
+            for (int d = lane; d < hd; d += 32) dst[d] = d < dv ? (BIAS ? il_from_f<TA>(il_to_f(x[d]) + bx[d]) : x[d]) : il_from_f<TA>(0.f);
         }
     }
 }
@@ -127,7 +141,7 @@ __global__ void qk_norm_store_kernel(const TA* proj, int ld, int q_off, int k_of
 IL_EXPORT int il_qk_norm_store(const void* proj, int act_kind, int ld, int q_off, int k_off, int v_off, int nh, int nkv, int dk, int dv, int hd,
                                const void* wq, const void* wk, int w_kind, float eps, float t_coef, int t_every, void* q_out,
                                const int* tok_pos, const int* tok_entry, const int* block_table, int bt_stride, void* cache, int page_size,
-                               int T, cudaStream_t stream) {
+                               int T, const float* bias, cudaStream_t stream) {
     if (T <= 0) return IL_OK;
     if (nh <= 0 || nkv <= 0 || dk <= 0 || dv <= 0 || hd < dk || hd < dv || page_size <= 0 || !wq || (k_off >= 0 && !wk)) return IL_BAD_ARG;
     const long long warps = (long long)T * (nh + (k_off >= 0 ? 2 * nkv : 0));
@@ -136,15 +150,20 @@ IL_EXPORT int il_qk_norm_store(const void* proj, int act_kind, int ld, int q_off
     if (act_kind != IL_F32 && act_kind != IL_BF16) return IL_BAD_ARG;
     const bool vec = ((ld | q_off | v_off | dk | dv | hd) & 3) == 0 && (k_off < 0 || (k_off & 3) == 0) &&
                      (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)cache) & 15) == 0;
-#define QN_GO(TA, VEC)                                                                                                                  \
-    IL_LAUNCH((qk_norm_store_kernel<TA, VEC>), (int)blocks, 128, 0, stream, (const TA*)proj, ld, q_off, k_off, v_off, nh, nkv, dk, dv, hd, wq, wk, \
-              w_kind, eps, t_coef, t_every, (TA*)q_out, tok_pos, tok_entry, block_table, bt_stride, (TA*)cache, page_size, T)
+#define QN_GO1(TA, VEC, BIAS)                                                                                                                  \
+    IL_LAUNCH((qk_norm_store_kernel<TA, VEC, BIAS>), (int)blocks, 128, 0, stream, (const TA*)proj, ld, q_off, k_off, v_off, nh, nkv, dk, dv, hd, wq, wk, \
+              w_kind, eps, t_coef, t_every, (TA*)q_out, tok_pos, tok_entry, block_table, bt_stride, (TA*)cache, page_size, T, bias)
+#define QN_GO(TA, VEC)                                                      \
+    do {                                                                    \
+        if (bias) QN_GO1(TA, VEC, true); else QN_GO1(TA, VEC, false);       \
+    } while (0)
     if (act_kind == IL_F32) {
         if (vec) QN_GO(float, 4); else QN_GO(float, 1);
     } else {
         if (vec) QN_GO(__nv_bfloat16, 4); else QN_GO(__nv_bfloat16, 1);
     }
 #undef QN_GO
+#undef QN_GO1
     IL_LAUNCH_CHECK();
     return IL_OK;
 }

@@ -259,17 +259,23 @@ __global__ void __launch_bounds__(256) norm_add_norm_kernel(float* resid, const 
         c[k] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (v < nv && !pos) c[k] = NanVec<TA, VW>::ld(branch + (size_t)r * H + v * VW);
     }
-    if (pos) {                                    // the rows of a token's choices, in the order of the choices
-        for (int i = 0; i < top; ++i) {
-            const TA* y = branch + (size_t)sp[i] * H;
-            const float w = sw[i];
+    if (pos) {                                    // the rows of a token's choices, added in the order of the choices, NR of them asked for at a time
+        constexpr int NR = MAXV <= 2 ? 4 : MAXV <= 4 ? 2 : 1;
+        for (int i0 = 0; i0 < top; i0 += NR) {
+            float4 t[NR][MAXV];
 #pragma unroll
-            for (int k = 0; k < MAXV; ++k) {
-                const int v = threadIdx.x + k * 256;
-                if (v < nv) {
-                    const float4 t = NanVec<TA, VW>::ld(y + v * VW);
-                    c[k].x = fmaf(w, t.x, c[k].x), c[k].y = fmaf(w, t.y, c[k].y), c[k].z = fmaf(w, t.z, c[k].z), c[k].w = fmaf(w, t.w, c[k].w);
+            for (int i = 0; i < NR; ++i)
+#pragma unroll
+                for (int k = 0; k < MAXV; ++k) {
+                    const int v = threadIdx.x + k * 256;
+                    t[i][k] = (i0 + i < top && v < nv) ? NanVec<TA, VW>::ld(branch + (size_t)sp[i0 + i] * H + v * VW) : make_float4(0.f, 0.f, 0.f, 0.f);
                 }
+#pragma unroll
+            for (int i = 0; i < NR; ++i) {
+                const float w = i0 + i < top ? sw[i0 + i] : 0.f;
+#pragma unroll
+                for (int k = 0; k < MAXV; ++k)
+                    c[k].x = fmaf(w, t[i][k].x, c[k].x), c[k].y = fmaf(w, t[i][k].y, c[k].y), c[k].z = fmaf(w, t[i][k].z, c[k].z), c[k].w = fmaf(w, t[i][k].w, c[k].w);
             }
         }
     }

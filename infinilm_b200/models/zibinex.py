@@ -144,7 +144,7 @@ def describe(cfg: ZibinexConfig) -> ModelSpec:
                                                   "gate_per": "head", "rot_part": m["rot_dim"], "position": pos}, f"l{i}.mix")
         else:
             mixer = PartSpec("qk_norm_attention", {"hidden": W, "n_heads": m["heads"], "n_kv_heads": m["kv_heads"], "qk_dim": m["dim"],
-                                                   "v_dim": m["vdim"], "scale": m["scale"], "eps": eps, "qkv_bias": True,
+                                                   "v_dim": m["vdim"], "scale": m["scale"], "eps": eps, "qkv_bias": True, "bias_in_norm": True,
                                                    "window": m["window"], "weights": "sigmoid", "distance_log": True}, f"l{i}.mix")
         ffn = ffn_norm = None
         branch_norms = {"mixer_branch_norm": norm(f"l{i}", "norm1b")}

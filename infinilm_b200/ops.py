@@ -361,12 +361,15 @@ def cast_rows(x: torch.Tensor, out: torch.Tensor) -> None:
 def qk_norm_store(proj: torch.Tensor, q_off: int, k_off: Optional[int], v_off: int, n_heads: int, n_kv_heads: int, qk_dim: int, v_dim: int,
                   head_dim: int, w_q: torch.Tensor, w_k: Optional[torch.Tensor], eps: float, temp_coef: float, temp_every: int,
                   q_out: torch.Tensor, tok_pos: torch.Tensor, tok_entry: torch.Tensor, block_table: torch.Tensor,
-                  cache: Optional[torch.Tensor], page_size: int) -> None:
+                  cache: Optional[torch.Tensor], page_size: int, bias: Optional[torch.Tensor] = None) -> None:
     """Per token and head: q / rms(q) * w_q (times 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1) if temp_every > 0)
     to `q_out` [T, heads * head_dim]; k / rms(k) * w_k to the K plane of the token's cache slot and the value columns (at
     `v_off`; the key columns themselves where the values are the keys as projected) to the V plane. Heads are laid out at
-    head_dim >= qk_dim, v_dim, the surplus zero. `k_off` None: the mixer has no keys of its own, only queries are normed."""
-    _need_cuda(proj, w_q, w_k, q_out, tok_pos, tok_entry, block_table, cache)
+    head_dim >= qk_dim, v_dim, the surplus zero. `k_off` None: the mixer has no keys of its own, only queries are normed.
+    `bias`: float32, one number per column of `proj`, added to q, k and v before anything else."""
+    _need_cuda(proj, w_q, w_k, q_out, tok_pos, tok_entry, block_table, cache, bias)
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != proj.shape[1] or not bias.is_contiguous()):
+        raise KernelError("qk_norm_store: bias float32, one per column of proj")
     T = proj.shape[0]
     has_k = k_off is not None
     if proj.stride(1) != 1 or q_off + n_heads * qk_dim > proj.shape[1] or (has_k and (k_off + n_kv_heads * qk_dim > proj.shape[1]
@@ -384,10 +387,10 @@ def qk_norm_store(proj: torch.Tensor, q_off: int, k_off: Optional[int], v_off: i
             raise KernelError("qk_norm_store: cache [pages,2,kv_heads,page,head_dim] of proj's dtype")
     f = _fn("qk_norm", "il_qk_norm_store", [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                             _c_void_p, _c_void_p, _c_int, _c_float, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p,
-                                            _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p])
+                                            _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p])
     _check(f(_ptr(proj), kind_of(proj.dtype), proj.stride(0), q_off, k_off if has_k else -1, v_off, n_heads, n_kv_heads, qk_dim, v_dim,
              head_dim, _ptr(w_q), _ptr(w_k), kind_of(w_q.dtype), eps, temp_coef, temp_every, _ptr(q_out), _ptr(tok_pos), _ptr(tok_entry),
-             _ptr(block_table), block_table.shape[1], _ptr(cache if has_k else None), page_size, T, _stream()), "qk_norm_store")
+             _ptr(block_table), block_table.shape[1], _ptr(cache if has_k else None), page_size, T, _ptr(bias), _stream()), "qk_norm_store")
 
 
 def qk_rows_norm_rope_store(proj: torch.Tensor, q_off: int, k_off: Optional[int], v_off: int, n_heads: int, n_kv_heads: int, qk_dim: int,
@@ -627,10 +630,14 @@ def attention_prefill_tc5(qkv: torch.Tensor, out: torch.Tensor, kv_map: torch.Te
                           entry_qstart: torch.Tensor, entry_kvlen: torch.Tensor, first_entry: int, n_entries: int,
                           n_tiles_total: int, page_size: int, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                           window: Optional[int], sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
-                          sigmoid: bool = False) -> None:
+                          sigmoid: bool = False, log_bias: Optional[torch.Tensor] = None) -> None:
     """The same attention as `attention_prefill`, on tcgen05 tensor cores with tensor memory; `kv_map` is the cache's
-    tensor map (`kv_tensor_map`). n_tiles_total = sum over the entries of ceil(q_len / (prefill_tc5_rows(head_dim) // (heads/kv_heads)))."""
-    _need_cuda(qkv, out, block_table, entry_qstart, entry_kvlen, sink, dist_bias)
+    tensor map (`kv_tensor_map`). `log_bias` (with `sigmoid`, instead of dist_bias): float32 [3, heads] - r1, r2 and an offset pb:
+    the scaled score of a key n positions back gets pb - r1 ln(1 + r2 n), computed as it is needed. n_tiles_total = sum over the entries of ceil(q_len / (prefill_tc5_rows(head_dim) // (heads/kv_heads)))."""
+    _need_cuda(qkv, out, block_table, entry_qstart, entry_kvlen, sink, dist_bias, log_bias)
+    if log_bias is not None and (not sigmoid or dist_bias is not None or log_bias.dtype != torch.float32 or tuple(log_bias.shape) != (3, n_heads)
+                                 or not log_bias.is_contiguous()):
+        raise KernelError("attention_prefill_tc5: log_bias float32 [3, heads], with sigmoid weights and without dist_bias")
     _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)
     if qkv.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
@@ -642,11 +649,11 @@ def attention_prefill_tc5(qkv: torch.Tensor, out: torch.Tensor, kv_map: torch.Te
     _contig("qkv", qkv), _contig("out", out), _contig("block_table", block_table)
     f = _fn("attn_prefill_tc5", "il_attn_prefill_tc5",
             [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p], defines={"HEAD_DIM": head_dim})
+             _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p], defines={"HEAD_DIM": head_dim})
     _check(f(_ptr(qkv), qkv.shape[1], _ptr(out), _c_void_p(kv_map.data_ptr() + 256), _ptr(block_table), block_table.shape[1],
              _ptr(entry_qstart), _ptr(entry_kvlen), page_size, first_entry, n_entries, n_tiles_total, n_heads, n_kv_heads,
              head_dim, scale, int(window or 0), _ptr(stream_status(qkv.device)), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1,
-             int(sigmoid), _stream()), "attention_prefill_tc5")
+             int(sigmoid), _ptr(log_bias), _stream()), "attention_prefill_tc5")
 
 
 SKINNY_MAX_ROWS = 16
@@ -1134,6 +1141,8 @@ def moe_sort(idx: torch.Tensor, n_experts: int, group_off: torch.Tensor, pos_of_
     f = _fn("moe", "il_moe_sort", [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p])
     _check(f(_ptr(idx), T * top, top, n_experts, _ptr(group_off), _ptr(pos_of_slot), _ptr(row_of_pos),
              _ptr(wt if wt_of_pos is not None else None), _ptr(wt_of_pos), _stream()), "moe_sort")
+    if T * top >= 4096:
+        count_launches(1)                         # the scattered half of a large sort is a kernel of its own
 
 
 def gather_rows(x: torch.Tensor, rows: torch.Tensor, out: torch.Tensor) -> None:

@@ -32,7 +32,9 @@ class PagedAttend:
     `chunk`: instead of a sliding window, runs of `chunk` positions counted from position 0 of the sequence; a query sees the
     keys of its own run up to itself (the kernels take it as a negative window). The cache keeps every page: a window's
     pages are given back behind it, a chunked layer's are not (another layer may read them).
-    `sigmoid`: no softmax - a visible key's weight is the sigmoid of its score (scaled, biased), not normalised over the keys."""
+    `sigmoid`: no softmax - a visible key's weight is the sigmoid of its score (scaled, biased), not normalised over the keys.
+    `log_bias`: float32 [3, heads] on the device or None - the numbers r1, r2, pb whose pb - r1 ln(1 + r2 n) `dist_bias` holds by
+    distance: a kernel that would rather compute than look up takes these (sigmoid weights on the tensor-memory prefill kernel)."""
 
     # The fast bfloat16 kernels take kernel pages of 16 keys (the cache manager lays larger pages out as runs of them)
     # and at most 64 query heads per kv head; anything else, and the whole float32 path, runs the plain kernel.
@@ -55,6 +57,7 @@ class PagedAttend:
         self.sigmoid = bool(sigmoid)
         self.sink: Optional[torch.Tensor] = None
         self.dist_bias: Optional[torch.Tensor] = None
+        self.log_bias: Optional[torch.Tensor] = None
 
     def fast_ok(self, page_size: int) -> bool:
         return (self.dtype == torch.bfloat16 and page_size == self.FAST_PAGE and self.nh // self.nkv <= self.FAST_MAX_GROUP
@@ -104,7 +107,8 @@ class PagedAttend:
             if tc5:
                 ops.attention_prefill_tc5(qkv, out, cache.tma_map, cache.block_table, ctx.entry_qstart, ctx.entry_kvlen,
                                           n_dec, E, n_tiles, cache.page_size, self.nh, self.nkv, self.hd, self.scale,
-                                          self.mask_arg, sink=self.sink, dist_bias=self.dist_bias, sigmoid=self.sigmoid)
+                                          self.mask_arg, sink=self.sink, dist_bias=self.dist_bias if self.log_bias is None else None,
+                                          sigmoid=self.sigmoid, log_bias=self.log_bias)
             else:
                 ops.attention_prefill(qkv, out, cache.storage, cache.block_table, ctx.entry_qstart, ctx.entry_kvlen,
                                       n_dec, E, n_tiles, cache.page_size, self.nh, self.nkv, self.hd, self.scale,

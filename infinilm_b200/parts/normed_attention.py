@@ -60,6 +60,7 @@ class QKNormAttention(Mixer):
     norm_over ("head", the default, or "projection": q.norm has heads * qk_dim entries, k.norm kv_heads * qk_dim),
     position (PartSpec of a rotary encoding, with norm_over "projection"), chunk (runs of that many positions, counted from the
     sequence's start; a query sees its own run) or window (a sliding window; its pages are given back behind it);
+    bias_in_norm (the projection's biases are added, in float32, by the kernel that norms; with a norm per head),
     weights ("softmax", the default, or "sigmoid"), distance_log (with a window, instead of distance_bias)."""
     graph_safe = True
     MAX_DISTANCES = 1 << 20                       # rows of an unrolled table by distance
@@ -125,7 +126,10 @@ class QKNormAttention(Mixer):
         self.o_proj = Linear(self.nh * self.dv, self.hidden, dtype)
         self.core = PagedAttend(dtype, self.nh, self.nkv, self.hd, self.scale, self.window, bool(p.get("plain_kernel", False)),
                                 str(p.get("prefill_kernel", "auto")), chunk=self.chunk, sigmoid=self.sigmoid)
-        self.w_q = self.w_k = None
+        self.bias_in_norm = bool(p.get("bias_in_norm", False)) and self.qkv_bias
+        if self.bias_in_norm and self.norm_rows:
+            raise ValueError("attention: biases join in the norm's kernel where the norm is per head")
+        self.w_q = self.w_k = self.bias = None
 
     def weight_specs(self) -> List[WeightSpec]:
         H = self.hidden
@@ -162,7 +166,10 @@ class QKNormAttention(Mixer):
         if self.qkv_bias:
             bs = [t[n + ".b"].float() for n in names]
             b = torch.cat(bs + [torch.zeros(self.n_proj_pad - sum(x.numel() for x in bs), dtype=torch.float32, device=dev)])
-        self.proj.set(torch.cat(ws, dim=0), b)
+        # bias_in_norm: the norm's kernel adds the biases, in float32, on its way to the cache; a bfloat16 product of many rows would
+        # need a pass over its rounded rows for them. (The 32-bit product adds them in its epilogue.)
+        self.bias = b if self.bias_in_norm and self.dtype == torch.bfloat16 else None
+        self.proj.set(torch.cat(ws, dim=0), None if self.bias is not None else b)
         self.o_proj.set(t["o"])
         self.w_q = t["q.norm"].to(torch.float32).contiguous()
         self.w_k = t["k.norm"].to(torch.float32).contiguous() if self.own_kv else None
@@ -177,6 +184,8 @@ class QKNormAttention(Mixer):
             if self.sigmoid:
                 table += t["pb"].double()[None, :]
             self.core.dist_bias = table.to(torch.float32).contiguous()
+            if self.sigmoid and self.dist_log:
+                self.core.log_bias = torch.stack([t["r1"].float(), t["r2"].float(), t["pb"].float()]).contiguous()
         if self.sink_zero:
             self.core.sink = torch.zeros(self.nh, dtype=torch.float32, device=dev)
         self.position.to_device(dev)
@@ -198,7 +207,7 @@ class QKNormAttention(Mixer):
         else:
             ops.qk_norm_store(proj, self.q_off, self.k_off, self.v_off if self.own_kv else 0, self.nh, self.nkv, self.dk, self.dv, hd,
                               self.w_q, self.w_k, self.eps, self.t_coef, self.t_every, q, ctx.tok_pos, ctx.tok_entry, cache.block_table,
-                              cache.storage if self.own_kv else None, cache.page_size)
+                              cache.storage if self.own_kv else None, cache.page_size, bias=self.bias)
         att = ctx.ws.rows("qna_att", T, self.nh * hd, self.dtype)
         self.core.run(q, att, ctx, cache)
         if self.gate or hd != self.dv:

@@ -199,6 +199,8 @@ def _run_attention(kernel, c, nh, nkv, hd, scale, window, dtype, splits=1):
                               16, nh, nkv, hd, scale, window, **kw)
     else:
         tpt = max(1, ops.prefill_tc5_rows(hd) // G)
+        if kernel == "tc5 log":                   # the bias by distance computed in the kernel
+            kw = dict(sigmoid=True, log_bias=torch.stack([c["r1"], c["r2"], c["pb"]]).contiguous().cuda())
         ops.attention_prefill_tc5(q, out, ops.kv_tensor_map(cache), bt, _i32(qstart), _i32(c["lens"]), 0, c["E"],
                                   sum((x + tpt - 1) // tpt for x in c["qlens"]), 16, nh, nkv, hd, scale, window, **kw)
     torch.cuda.synchronize()
@@ -211,7 +213,8 @@ WINDOWS = [20, 16, 17, 1, 2, 90, 300]
 
 @pytest.mark.parametrize("kernel,dtype,nh,nkv,hd", [("plain", "float32", 3, 1, 40), ("plain", "bfloat16", 6, 3, 48), ("prefill", "bfloat16", 6, 3, 48),
                                                     ("prefill", "bfloat16", 8, 8, 80), ("tc5", "bfloat16", 4, 2, 64), ("tc5", "bfloat16", 9, 1, 128),
-                                                    ("tc5", "bfloat16", 4, 1, 256)])
+                                                    ("tc5", "bfloat16", 4, 1, 256), ("tc5 log", "bfloat16", 4, 2, 64), ("tc5 log", "bfloat16", 9, 1, 128),
+                                                    ("tc5 log", "bfloat16", 4, 1, 256)])
 def test_sigmoid_weights_over_portions(cuda_device, kernel, dtype, nh, nkv, hd):
     """Portions that start and end anywhere, with one key made to stand out: the oldest key a window shows, the one before it,
     and keys at page borders. A query that may see the key follows it; one that may not must not. (Without a marked key an
@@ -236,7 +239,7 @@ def test_sigmoid_weights_of_single_tokens(cuda_device, kernel, dtype, nh, nkv, h
             _close(got, _attn_reference(c, nh, nkv, 0.2, size, dtype), dtype, f"{kernel} window {size}, marked {mk}")
 
 
-@pytest.mark.parametrize("kernel,hd", [("plain", 64), ("prefill", 64), ("tc5", 64), ("decode", 64)])
+@pytest.mark.parametrize("kernel,hd", [("plain", 64), ("prefill", 64), ("tc5", 64), ("tc5 log", 64), ("decode", 64)])
 def test_extreme_scores_and_masked_garbage(cuda_device, kernel, hd):
     """Scores far beyond where the exponential overflows (weights 0 and 1), with keys of neighbours' huge values outside the
     window: a masked key's weight is zero, not small."""
@@ -252,6 +255,28 @@ def test_extreme_scores_and_masked_garbage(cuda_device, kernel, hd):
         n = c["lens"][e]
         c["v"][e][: n - 10] = 0.0
     _close(got, _attn_reference(c, 2, 1, 1.0, 10, "bfloat16" if kernel != "plain" else "float32"), "bfloat16", kernel)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("nh,nkv,dk,dv", [(4, 2, 32, 16), (3, 1, 20, 12), (2, 2, 7, 40)])
+def test_norm_per_head_adds_the_biases_first(cuda_device, dtype, nh, nkv, dk, dv):
+    from infinilm_b200 import ops
+    g = torch.Generator().manual_seed(dk)
+    dt = DT[dtype]
+    T, hd = 19, (max(dk, dv) + 15) // 16 * 16
+    nq, nk, nv = nh * dk, nkv * dk, nkv * dv
+    ld = (nq + nk + nv + 7) // 8 * 8
+    proj, bias = torch.randn(T, ld, generator=g).to(dt), torch.randn(ld, generator=g) * 2
+    wq, wk = 1.0 + 0.2 * torch.randn(dk, generator=g), 1.0 + 0.2 * torch.randn(dk, generator=g)
+    cache, q_out = torch.zeros(2, 2, nkv, 16, hd, dtype=dt, device="cuda"), torch.empty(T, nh * hd, dtype=dt, device="cuda")
+    ops.qk_norm_store(proj.cuda(), 0, nq, nq + nk, nh, nkv, dk, dv, hd, wq.cuda(), wk.cuda(), 1e-4, 0.0, 0, q_out, _i32(list(range(T))), _i32([0] * T),
+                      _i32([[1, 0]]), cache, 16, bias=bias.cuda())
+    x = proj.double() + bias.double()
+    tol = 2e-6 if dtype == "float32" else 6e-3
+    _close(q_out.view(T, nh, hd)[:, :, :dk], P.rms_norm(x[:, :nq].view(T, nh, dk), wq.double(), 1e-4), dtype, "q", tol)
+    rows = torch.cat([cache[1], cache[0]], dim=2)[:, :, :T].transpose(1, 2)          # [plane, T, kv heads, hd]
+    _close(rows[0, :, :, :dk], P.rms_norm(x[:, nq:nq + nk].view(T, nkv, dk), wk.double(), 1e-4), dtype, "k", tol)
+    _close(rows[1, :, :, :dv], x[:, nq + nk:nq + nk + nv].view(T, nkv, dv), dtype, "v", tol)
 
 
 # ---- the clamped gate ---------------------------------------------------------------------------------------------------------------
@@ -356,6 +381,18 @@ def test_gate_per_group(cuda_device, dtype, M, G, N, K):
     ops.gemm_grouped(heads, w.cuda(), out, gate=gate.cuda()[:, 2:2 + G])
     want = torch.einsum("mgk,gnk->mgn", a[:, :G * (K + 16)].view(M, G, K + 16)[:, :, :K].double(), w.double())
     _close(out, want * torch.sigmoid(gate[:, 2:2 + G].double())[:, :, None], dtype, "gated", 1e-5 if dtype == "float32" else 1e-2)
+
+
+@pytest.mark.parametrize("vdim,hd,ldg", [(24, 24, 9), (64, 64, 4), (20, 32, 4), (16, 48, 5)])
+def test_head_gate_in_pieces_and_by_columns(cuda_device, vdim, hd, ldg):
+    from infinilm_b200 import ops
+    g = torch.Generator().manual_seed(vdim)
+    T, nh = 37, 3
+    y, gate = torch.randn(T, nh * hd, generator=g).to(torch.bfloat16), torch.randn(T, ldg, generator=g).to(torch.bfloat16)
+    out = torch.empty(T, nh * vdim, dtype=torch.bfloat16, device="cuda")
+    ops.head_gate(y.cuda(), hd, gate.cuda(), 1, out, nh, vdim)
+    want = y.double().view(T, nh, hd)[:, :, :vdim] * torch.sigmoid(gate.double()[:, 1:1 + nh])[:, :, None]
+    _close(out.view(T, nh, vdim), want, "bfloat16", "gated", 6e-3)
 
 
 @pytest.mark.parametrize("nh,d,rd,e,r", [(4, 32, 16, 24, 48), (2, 64, 32, 64, 96), (4, 64, 64, 64, 192)])
