@@ -180,6 +180,7 @@ class SequenceCache:
     seq_id: object
     length: int = 0                               # tokens whose keys/values (or state) are in the cache
     tables: Dict[int, List[int]] = field(default_factory=dict)   # group -> page id per page index (-1: given back)
+    given_back: Dict[int, int] = field(default_factory=dict)     # windowed group -> pages of its table given back so far
     state_slot: int = 0
     fresh_state: bool = True                      # no step has run yet: state groups start from the zero state
     open: bool = True
@@ -324,10 +325,13 @@ class CacheManager:
             if grp.need.window is None:
                 continue
             first = self._first_needed_page(grp, new_len)
-            for idx in range(min(first, len(tbl))):
+            done, first = seq.given_back.get(g, 0), min(first, len(tbl))
+            for idx in range(done, first):        # (a long request's pages are not looked at again step after step)
                 if tbl[idx] >= 0:
                     grp.pool.free(tbl[idx])
                     tbl[idx] = -1
+            if first > done:
+                seq.given_back[g] = first
 
     def close(self, seq: SequenceCache) -> None:
         """The request is finished: all it holds is given back."""
@@ -337,6 +341,7 @@ class CacheManager:
                 if p >= 0:
                     self.groups[g].pool.free(p)
             tbl.clear()
+        seq.given_back.clear()
         self.slots.free(seq.state_slot)
         seq.open = False
         del self.live[seq.seq_id]

@@ -227,14 +227,23 @@ class StepRunner:
         self.h2d_bytes += 4 * n
         gs.graph.replay()
         ops.count_launches(gs.n_kernels)
-        for s_ in seqs:                           # what CacheManager.commit does for a request without a window
-            s_.length += 1
+        for w in self._windows():                 # where a window leaves a page behind, the page goes back ...
+            gone = lens + 1 - w + 1               # first position a later query can still see, at the length to come
+            for i in np.flatnonzero((gone > 0) & (gone % ps == 0)):
+                if seqs[i].length == int(lens[i]):
+                    cache.commit(seqs[i], int(lens[i]) + 1)
+        for s_, n_ in zip(seqs, lens.tolist()):   # ... and this is what CacheManager.commit does for every other request
+            s_.length = n_ + 1
         last.lens = lens + 1
         self._last_decode = last
         self.steps_run += 1
         self.tokens_run += E
         self.fast_steps += 1
         return gs.logits[:E]
+
+    def _windows(self) -> List[int]:
+        """The window sizes of the cache's groups, each once."""
+        return sorted({grp.need.window for grp in self.cache.groups if grp.need.kind == "paged_kv" and grp.need.window is not None})
 
     # -- a step's entries as columns, checked --------------------------------------------------------
     def _columns(self, entries: Sequence[StepEntry], device_tokens: Optional[torch.Tensor]) -> "_Columns":
@@ -468,7 +477,7 @@ class StepRunner:
                 gs.graph.replay()
                 ops.count_launches(gs.n_kernels)
                 self.portion_replays += n_decode != E
-                if n_decode == E and not any(grp.need.kind == "paged_kv" and grp.need.window is not None for grp in groups):
+                if n_decode == E:
                     # the next step may be the same requests with one more token each: keep what it can start from
                     self._last_decode = _DecodeBatch(
                         seqs=seqs, gs=gs, E=E, Ep=Ep, widths=dict(widths), mirror=h[:off].copy(), lens=start + 1,

@@ -238,15 +238,19 @@ def test_a_far_token_reaches_the_end(cuda_device, dtype):
     eng.synchronize()
 
 
-def test_windows_pages_are_given_back(cuda_device):
+@pytest.mark.parametrize("graphs", [False, True])
+def test_windows_pages_are_given_back(cuda_device, graphs):
     """A model of windowed layers alone decodes far longer than its pool could hold: the pages behind the window come back."""
     raw = ZIBINEX["a"]()
     raw["layers"] = [raw["layers"][1], raw["layers"][4]]
     w = make_weights(raw, 8, clear_choices=True)
     eng = _engine(raw, w, "bfloat16", num_pages=6)
+    if graphs:                                    # a replayed step made from the step before gives pages back as any other
+        eng.enable_graphs()
     ids = token_ids(400, raw["vocab"], 3)
     got = _run_cut(eng, ids, [40] + [1] * 300 + [33, 27])
     _check(got, _plain(raw, w, ids), "bfloat16", "400 tokens through 6 pages a group")
+    assert not graphs or eng.runner.fast_steps > 200
     eng.synchronize()
     eng.cache.check_invariants()
 
@@ -331,3 +335,44 @@ def test_trace_runner_as_a_process(cuda_device, tmp_path):
             want = torch.stack([ref[rid][0][pos] for rid, pos in rows])
             margin = torch.stack([torch.cummin(ref[rid][1], 0).values[pos] for rid, pos in rows])
             _check(got, (want, margin), dtype, f"trace step {n} ({dtype})", cum=False)
+
+
+@pytest.mark.parametrize("name,seed", [("a", 0), ("d", 3)])
+def test_a_batch_decodes_in_replayed_steps_past_its_windows(cuda_device, name, seed):
+    """Three unequal requests decode side by side in replayed steps, each made from the step before, while every one's windows
+    leave pages behind at steps of its own and others take those pages; a fourth joins in between."""
+    from infinilm_b200.engine import StepEntry
+    raw = ZIBINEX[name]()
+    w = _weights(name, seed, "bfloat16")
+    eng = _engine(raw, w, "bfloat16", num_pages=36)
+    eng.enable_graphs()
+    req = {k: token_ids(n, raw["vocab"], 60 + n) for k, n in (("p", 150), ("q", 131), ("r", 137), ("s", 40))}
+    first = {"p": 30, "q": 11, "r": 17, "s": 20}
+    seqs, at, out = {}, {}, {k: [] for k in req}
+
+    def step(who):
+        ent = [StepEntry(seqs[k], req[k][at[k]:at[k] + n], list(range(n)) if n == 1 else [n - 1]) for k, n in who]
+        lg = eng.step(ent).clone()
+        for i, (k, n) in enumerate(who):
+            at[k] += n
+            out[k].append((at[k] - 1, lg[i]))
+    for k in "pqr":
+        seqs[k], at[k] = eng.open(k), 0
+        step([(k, first[k])])
+    for n in range(60):
+        step([(k, 1) for k in "pqr"])
+        eng.cache.check_invariants()
+    seqs["s"], at["s"] = eng.open("s"), 0
+    step([("p", 1), ("s", 20), ("q", 1), ("r", 1)])
+    for n in range(20):
+        step([(k, 1) for k in "pqrs"])
+    eng.close(seqs.pop("s"))
+    for n in range(39):
+        step([(k, 1) for k in "pqr"])
+        eng.cache.check_invariants()
+    assert eng.runner.fast_steps > 90
+    for k in req:
+        lg, margin = _plain(raw, w, req[k])
+        pos = torch.tensor([p for p, _ in out[k]])
+        _check(torch.stack([x for _, x in out[k]]), (lg[pos], torch.cummin(margin, 0).values[pos]), "bfloat16", f"request {k}", cum=False)
+    eng.synchronize()
