@@ -248,14 +248,15 @@ __global__ void __launch_bounds__(WARPS * 32) moe_select_kernel(const float* __r
 // fused kernel below reads what its own warps have just written.) `wt_of_pos` (or null) receives every place's weight: where a
 // choice's weight belongs to the expert's input, the products take it as a factor per place. row_of_pos null: a kernel behind this
 // one fills in what lies in the order of the places.
+template <int SL>
 __device__ __forceinline__ void moe_sort_body(int* sh, const int* idx, int n_slots, int top, int E, int* __restrict__ group_off,
                                               int* __restrict__ pos_of_slot, int* __restrict__ row_of_pos, const float* wt, float* __restrict__ wt_of_pos) {
     int* cnt = sh;
     int* cur = sh + E;
     for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
     __syncthreads();
-    // (SL slots of a thread asked for at a time: one after the other they are a chain of round trips to memory)
-    constexpr int SL = 8;
+    // (SL slots of a thread asked for at a time: one after the other the slots of a long portion are a chain of round trips to
+    // memory; a decode step has at most one a thread)
     for (int i0 = threadIdx.x; i0 < n_slots; i0 += SL * blockDim.x) {
         int e[SL];
 #pragma unroll
@@ -316,12 +317,13 @@ __global__ void moe_places_kernel(const int* pos_of_slot, int n_slots, int top, 
     if (wt_of_pos) wt_of_pos[p] = wt[i];
 }
 
+template <int SL>
 __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* idx, int n_slots, int top, int E, int* __restrict__ group_off,
                                                         int* __restrict__ pos_of_slot, int* __restrict__ row_of_pos, const float* wt,
                                                         float* __restrict__ wt_of_pos) {
     extern __shared__ int sh[];                   // [E] counts, then [E] cursors
     il_pdl_begin();
-    moe_sort_body(sh, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
+    moe_sort_body<SL>(sh, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
 }
 
 // ---- the router of a decode step (a few bfloat16 rows) as two short kernels --------------------------------------------
@@ -395,7 +397,7 @@ __global__ void __launch_bounds__(1024) moe_select_sort_kernel(const float* z, i
         __syncwarp();
     }
     __syncthreads();                              // the choices, written to memory by this block's warps, are read below
-    moe_sort_body(reinterpret_cast<int*>(sm + (size_t)32 * E), idx, T * top, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
+    moe_sort_body<1>(reinterpret_cast<int*>(sm + (size_t)32 * E), idx, T * top, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
 }
 
 __device__ __forceinline__ float4 ld4c(const float* p) { return *reinterpret_cast<const float4*>(p); }
@@ -630,10 +632,10 @@ IL_EXPORT int il_moe_sort(const int* idx, int n_slots, int top, int E, int* grou
     const size_t smem = (size_t)2 * E * sizeof(int);
     if (smem > 48 * 1024) return IL_UNSUPPORTED;
     if (n_slots >= 4096) {
-        IL_LAUNCH(moe_sort_kernel, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, (int*)nullptr, (const float*)nullptr, (float*)nullptr);
+        IL_LAUNCH(moe_sort_kernel<8>, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, (int*)nullptr, (const float*)nullptr, (float*)nullptr);
         IL_LAUNCH(moe_places_kernel, (n_slots + 255) / 256, 256, 0, stream, (const int*)pos_of_slot, n_slots, top, row_of_pos, wt, wt_of_pos);
     } else {
-        IL_LAUNCH(moe_sort_kernel, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
+        IL_LAUNCH(moe_sort_kernel<1>, 1, 1024, smem, stream, idx, n_slots, top, E, group_off, pos_of_slot, row_of_pos, wt, wt_of_pos);
     }
     IL_LAUNCH_CHECK();
     return IL_OK;
