@@ -24,7 +24,7 @@
 //
 // Two kinds of weights. Softmax, as above; or - the template's SIG - every visible key's own sigmoid of its (scaled, biased)
 // score, with no normalisation over the keys: the running maximum then stays 0, nothing is rescaled, the splits' partials are
-// plain sums and the merge adds them.
+// plain sums and the merge adds them. With softmax weights the score may be soft-capped (CAP): cap * tanh(scaled score / cap).
 #include <cuda.h>
 #include <cstring>
 
@@ -164,14 +164,14 @@ __device__ __forceinline__ void ad_merge_row(float* fs, float* comb, const float
 // (qkv, and o_part / ml_part in the merge, are written by the kernel before and read after a wait that is not the
 // kernel's first statement: they are not declared __restrict__, so that no load of them is treated as read-only
 // data and scheduled above the wait.)
-template <bool SIG>
+template <bool SIG, bool CAP>
 __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_kernel(
     const __nv_bfloat16* qkv, int row_stride, const __nv_bfloat16* __restrict__ cache,
     const int* __restrict__ block_table, int bt_stride, const int* __restrict__ entry_kvlen, int nh, int nkv,
     float scale_log2, int window, int pages_per_split, int n_splits, float* __restrict__ o_part,
     float* __restrict__ ml_part, const __grid_constant__ CUtensorMap kv_map, const __grid_constant__ CUtensorMap kv_page_map,
     int use_tma, int* __restrict__ status, __nv_bfloat16* __restrict__ out_direct, const float* __restrict__ sink,
-    const float* __restrict__ dist_bias, int dist_far) {
+    const float* __restrict__ dist_bias, int dist_far, float cap_log2) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     // Lengths, block tables and the pages of earlier tokens do not come from the kernel before this one (it writes q and
@@ -307,7 +307,7 @@ __global__ void __launch_bounds__(AD_WARPS * 32) attn_decode_kernel(
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int key = key0 + nt * 8 + (j & 1);
-                float v = s[nt][j] * scale_log2;
+                float v = CAP ? il_cap_log2_fast(s[nt][j], scale_log2, cap_log2) : s[nt][j] * scale_log2;
                 if (dist_bias) v += db_near ? db_row[j >> 1][max(0, min(kvlen - 1 - key, dist_far)) * nh] * 1.4426950408889634f : db_far[j >> 1];
                 if (SIG) s[nt][j] = (key >= lo && key < hi) ? il_sigmoid_log2_fast(v) : 0.f;
                 else s[nt][j] = (key >= lo && key < hi) ? v : -INFINITY;
@@ -524,7 +524,7 @@ static int ad_launch(const void* qkv, int row_stride, void* out, const void* cac
                      const int* entry_kvlen, int n_decode, int nh, int nkv, float scale, int window, int pages_per_split,
                      int n_splits, float* o_part, float* ml_part, cudaStream_t stream, const CUtensorMap* kv_map = nullptr,
                      int* status = nullptr, const float* sink = nullptr, int v_is_k = 0, const float* dist_bias = nullptr,
-                     int dist_far = 0, int sigmoid = 0) {
+                     int dist_far = 0, int sigmoid = 0, float cap = 0.f) {
     static CUtensorMap no_map;                    // passed when there is no map: the kernel does not look at it
     int use_tma = (AD_TMA_OK && kv_map && status) ? 1 : 0;
     auto filled = [&](int i) {                    // maps behind the first are all zero where the driver did not take them
@@ -541,19 +541,24 @@ static int ad_launch(const void* qkv, int row_stride, void* out, const void* cac
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev >= 0 && dev < 64 && !attr_set[dev]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_decode_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_decode_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_decode_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM);
         if (e != cudaSuccess) return 1000 + (int)e;
         attr_set[dev] = true;
     }
     const int G = nh / nkv, row_tiles = (G + 15) / 16;
     dim3 grid(n_splits, nkv * row_tiles, n_decode);
-#define AD_GO(SIG)                                                                                                                           \
-    IL_LAUNCH(attn_decode_kernel<SIG>, grid, AD_WARPS * 32, smem_bytes, stream, (const __nv_bfloat16*)qkv, row_stride,                       \
-              (const __nv_bfloat16*)cache, block_table, bt_stride, entry_kvlen, nh, nkv, scale * 1.4426950408889634f, window, pages_per_split, \
+#define AD_GO(SIG, CAP)                                                                                                                      \
+    IL_LAUNCH((attn_decode_kernel<SIG, CAP>), grid, AD_WARPS * 32, smem_bytes, stream, (const __nv_bfloat16*)qkv, row_stride,                       \
+              (const __nv_bfloat16*)cache, block_table, bt_stride, entry_kvlen, nh, nkv, k_scale, window, pages_per_split,               \
               n_splits, o_part, ml_part, use_tma ? *kv_map : no_map, page_map, use_tma, status,                                              \
-              n_splits == 1 ? (__nv_bfloat16*)out : (__nv_bfloat16*)nullptr, sink, dist_bias, dist_far)
-    if (sigmoid) AD_GO(true); else AD_GO(false);
+              n_splits == 1 ? (__nv_bfloat16*)out : (__nv_bfloat16*)nullptr, sink, dist_bias, dist_far, cap * 1.4426950408889634f)
+    // a capped score's factor goes into the tanh's argument (il_cap_log2_fast), any other's into the exponent
+    const float k_scale = (cap > 0.f ? 2.f * scale / cap : scale) * 1.4426950408889634f;
+    if (sigmoid) AD_GO(true, false);
+    else if (cap > 0.f) AD_GO(false, true);
+    else AD_GO(false, false);
 #undef AD_GO
     if (n_splits == 1) {                          // every row is final as the attention kernel leaves it: no merge
         IL_LAUNCH_CHECK();
@@ -580,8 +585,8 @@ static int ad_resident_blocks(int v_is_k) {
     const int k = (v_is_k && AD_TMA_OK) ? 1 : 0, smem = k ? AD_SMEM_K : AD_SMEM;
     if (cached[k][dev]) return cached[k][dev];
     int per_sm = 0, sms = 0;
-    if (cudaFuncSetAttribute(attn_decode_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM) != cudaSuccess ||
-        cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attn_decode_kernel<false>, AD_WARPS * 32, smem) != cudaSuccess ||
+    if (cudaFuncSetAttribute(attn_decode_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AD_SMEM) != cudaSuccess ||
+        cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, attn_decode_kernel<false, false>, AD_WARPS * 32, smem) != cudaSuccess ||
         cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) {
         cudaGetLastError();
         return 0;
@@ -599,15 +604,16 @@ IL_EXPORT int il_attn_decode(const void* qkv, int row_stride, void* out, const v
                              int bt_stride, const int* entry_kvlen, int page_size, int n_decode, int nh, int nkv, int hd,
                              float scale, int window, int pages_per_split, int n_splits, float* o_part, float* ml_part,
                              const void* kv_map, int* status, const float* sink, int v_is_k, const float* dist_bias, int dist_far,
-                             int sigmoid, cudaStream_t stream) {
+                             int sigmoid, float cap, cudaStream_t stream) {
     if (n_decode <= 0) return IL_OK;
+    if (cap > 0.f && (sigmoid || dist_bias)) return IL_BAD_ARG;
     if (sigmoid && sink) return IL_BAD_ARG;       // a sink is a term of a softmax's denominator
     if (dist_bias && (dist_far < 0 || (long long)(dist_far + 1) * nh > 0x7fffffffLL)) return IL_BAD_ARG;
     if (hd != HEAD_DIM || page_size != AD_PAGE) return IL_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || pages_per_split < 0 || n_splits <= 0) return IL_BAD_ARG;
     if (n_splits > AD_MAX_SPLITS) return IL_UNSUPPORTED;
     return ad_launch(qkv, row_stride, out, cache, block_table, bt_stride, entry_kvlen, n_decode, nh, nkv, scale, window,
-                     pages_per_split, n_splits, o_part, ml_part, stream, (const CUtensorMap*)kv_map, status, sink, v_is_k, dist_bias, dist_far, sigmoid);
+                     pages_per_split, n_splits, o_part, ml_part, stream, (const CUtensorMap*)kv_map, status, sink, v_is_k, dist_bias, dist_far, sigmoid, cap);
 }
 
 // Writes four tensor maps (4 x 128 bytes at `out_maps`) of one layer's cache, [pages][2][kv heads][16][head_dim] bfloat16:

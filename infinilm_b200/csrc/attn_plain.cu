@@ -10,16 +10,16 @@
 // With `dist_bias` (f32 [dist_far + 1][heads]) the scaled score of a key n positions back gets dist_bias[min(n, dist_far)][head]
 // added: a learned bias by distance that is constant from dist_far on.
 // SIG: no softmax - a visible key's weight is the sigmoid of its (scaled, biased) score, and the weights are not
-// normalised over the keys.
+// normalised over the keys. CAP: the scaled score s becomes cap * tanh(s / cap) (a soft cap; the sink is not capped).
 #include "common.cuh"
 
 // A lane holds head_dim / 32 elements of the query and of the output: 8 (head_dim <= 256) or 32 (<= 1024).
-template <typename TA, int AP_MAX_PER_LANE, bool SIG>
+template <typename TA, int AP_MAX_PER_LANE, bool SIG, bool CAP>
 __global__ void attn_plain_kernel(const TA* __restrict__ qkv, int row_stride, TA* __restrict__ out,
                                   const TA* __restrict__ cache, const int* __restrict__ block_table, int bt_stride,
                                   const int* __restrict__ tok_pos, const int* __restrict__ tok_entry, int page_size,
                                   int nh, int nkv, int hd, float scale, int window, const float* __restrict__ sink,
-                                  const float* __restrict__ dist_bias, int dist_far) {
+                                  const float* __restrict__ dist_bias, int dist_far, float cap) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int j = blockIdx.y * (blockDim.x >> 5) + warp;
     const int t = blockIdx.x;
@@ -50,6 +50,7 @@ __global__ void attn_plain_kernel(const TA* __restrict__ qkv, int row_stride, TA
             if (d < hd) dot += q[r] * il_to_f(krow[d]);
         }
         dot = il_warp_sum(dot) * scale;
+        if (CAP) dot = cap * tanhf(dot / cap);
         if (dist_bias) dot += dist_bias[(size_t)min(pos - kp, dist_far) * nh + j];
         if constexpr (SIG) {
             const float w = 1.f / (1.f + expf(-dot));
@@ -84,19 +85,21 @@ __global__ void attn_plain_kernel(const TA* __restrict__ qkv, int row_stride, TA
 IL_EXPORT int il_attn_plain(const void* qkv, int act_kind, int row_stride, void* out, const void* cache,
                             const int* block_table, int bt_stride, const int* tok_pos, const int* tok_entry,
                             int page_size, int T, int nh, int nkv, int hd, float scale, int window,
-                            const float* sink, const float* dist_bias, int dist_far, int sigmoid, cudaStream_t stream) {
+                            const float* sink, const float* dist_bias, int dist_far, int sigmoid, float cap, cudaStream_t stream) {
     if (T <= 0) return IL_OK;
-    if ((dist_bias && dist_far < 0) || (sigmoid && sink)) return IL_BAD_ARG;
+    if ((dist_bias && dist_far < 0) || (sigmoid && sink) || (cap > 0.f && (sigmoid || dist_bias))) return IL_BAD_ARG;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || hd <= 0 || page_size <= 0) return IL_BAD_ARG;
     if (hd > 1024) return IL_UNSUPPORTED;
     const int warps = 4;
     dim3 grid(T, (nh + warps - 1) / warps);
-#define AP_LAUNCH1(TA, N, S)                                                                                                                \
-    attn_plain_kernel<TA, N, S><<<grid, warps * 32, 0, stream>>>((const TA*)qkv, row_stride, (TA*)out, (const TA*)cache, block_table, bt_stride, \
-                                                              tok_pos, tok_entry, page_size, nh, nkv, hd, scale, window, sink, dist_bias, dist_far)
+#define AP_LAUNCH1(TA, N, S, C)                                                                                                             \
+    attn_plain_kernel<TA, N, S, C><<<grid, warps * 32, 0, stream>>>((const TA*)qkv, row_stride, (TA*)out, (const TA*)cache, block_table, bt_stride, \
+                                                              tok_pos, tok_entry, page_size, nh, nkv, hd, scale, window, sink, dist_bias, dist_far, cap)
 #define AP_LAUNCH(TA, N)                                            \
     do {                                                            \
-        if (sigmoid) AP_LAUNCH1(TA, N, true); else AP_LAUNCH1(TA, N, false); \
+        if (sigmoid) AP_LAUNCH1(TA, N, true, false);                \
+        else if (cap > 0.f) AP_LAUNCH1(TA, N, false, true);         \
+        else AP_LAUNCH1(TA, N, false, false);                       \
     } while (0)
     if (act_kind == IL_F32) {
         if (hd <= 256) AP_LAUNCH(float, 8); else AP_LAUNCH(float, 32);

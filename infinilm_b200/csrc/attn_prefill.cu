@@ -9,6 +9,7 @@
 //   wholly behind its window, are skipped by that warp.
 //
 //   SIG: no softmax - a visible key's weight is the sigmoid of its (scaled, biased) score, not normalised over the keys.
+//   CAP: softmax over soft-capped scores, cap * tanh(scaled score / cap).
 //
 //   grid (tiles, kv heads). Tiles are numbered over the entries [first_entry, n_entries) in
 //   order; a block finds its entry by walking entry_qstart.
@@ -30,14 +31,15 @@ __device__ __forceinline__ float ap_ex2(float x) {
     return y;
 }
 
-template <bool SIG>
+template <bool SIG, bool CAP>
 __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
     const __nv_bfloat16* __restrict__ qkv, int row_stride, __nv_bfloat16* __restrict__ out,
     const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_table, int bt_stride,
     const int* __restrict__ entry_qstart, const int* __restrict__ entry_kvlen, int first_entry, int n_entries, int nh,
-    int nkv, float scale_log2, int window, int tpt, const float* __restrict__ sink, const float* __restrict__ dist_bias, int dist_far,
-    float inv_scale) {
+    int nkv, float k_scale, int window, int tpt, const float* __restrict__ sink, const float* __restrict__ dist_bias, int dist_far,
+    float inv_scale, float cap_log2) {
     extern __shared__ __align__(16) unsigned char smem[];
+    const float scale_log2 = CAP ? 1.f : k_scale; // (capped scores leave il_cap_log2_fast in base 2 already; k_scale is then its factor)
     const int G = nh / nkv;
     const int g = blockIdx.y;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -187,6 +189,7 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
                     const int h = j >> 1;
                     const int key = k0 + nt * 8 + (lane & 3) * 2 + (j & 1);
                     if (dist_bias) s[p][nt][j] += db_near ? db_row[h][max(0, min(rpos[h] - key, dist_far)) * nh] * inv_scale : db_far[h];
+                    if (CAP) s[p][nt][j] = il_cap_log2_fast(s[p][nt][j], k_scale, cap_log2);
                     if (need_mask) {
                         if (!(key <= rpos[h] && key >= rlo[h])) s[p][nt][j] = -INFINITY;
                     }
@@ -260,9 +263,10 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prefill_kernel(
 IL_EXPORT int il_attn_prefill(const void* qkv, int row_stride, void* out, const void* cache, const int* block_table,
                               int bt_stride, const int* entry_qstart, const int* entry_kvlen, int page_size,
                               int first_entry, int n_entries, int n_tiles_total, int nh, int nkv, int hd, float scale,
-                              int window, const float* sink, const float* dist_bias, int dist_far, int sigmoid, cudaStream_t stream) {
+                              int window, const float* sink, const float* dist_bias, int dist_far, int sigmoid, float cap, cudaStream_t stream) {
     if (n_tiles_total <= 0 || first_entry >= n_entries) return IL_OK;
     if (dist_bias && (dist_far < 0 || !(scale > 0.f) || (long long)(dist_far + 1) * nh > 0x7fffffffLL)) return IL_BAD_ARG;
+    if (cap > 0.f && (sigmoid || dist_bias)) return IL_BAD_ARG;
     if (sigmoid && (sink || !(scale > 0.f))) return IL_BAD_ARG;      // (a masked score is -inf before it is scaled)
     if (hd != HEAD_DIM || page_size != AP_PAGE) return IL_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) return IL_BAD_ARG;
@@ -270,16 +274,17 @@ IL_EXPORT int il_attn_prefill(const void* qkv, int row_stride, void* out, const 
     if (G > AP_ROWS) return IL_UNSUPPORTED;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AP_SMEM);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AP_SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AP_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AP_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AP_SMEM);
         if (e != cudaSuccess) return 1000 + (int)e;
         attr_set = true;
     }
     dim3 grid(n_tiles_total, nkv);
-    (sigmoid ? attn_prefill_kernel<true> : attn_prefill_kernel<false>)<<<grid, AP_WARPS * 32, AP_SMEM, stream>>>(
+    (sigmoid ? attn_prefill_kernel<true, false> : cap > 0.f ? attn_prefill_kernel<false, true> : attn_prefill_kernel<false, false>)<<<grid, AP_WARPS * 32, AP_SMEM, stream>>>(
         (const __nv_bfloat16*)qkv, row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)cache, block_table, bt_stride,
-        entry_qstart, entry_kvlen, first_entry, n_entries, nh, nkv, scale * 1.4426950408889634f, window, AP_ROWS / G, sink, dist_bias, dist_far,
-        1.f / scale);
+        entry_qstart, entry_kvlen, first_entry, n_entries, nh, nkv, (cap > 0.f ? 2.f * scale / cap : scale) * 1.4426950408889634f, window, AP_ROWS / G, sink,
+        dist_bias, dist_far, 1.f / scale, cap * 1.4426950408889634f);
     IL_LAUNCH_CHECK();
     return IL_OK;
 }

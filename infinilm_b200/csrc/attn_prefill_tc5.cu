@@ -35,6 +35,8 @@
 //   LOGB (with SIG): the bias by distance is pb_h - r1_h ln(1 + r2_h n), made here of three numbers per head instead of read
 //   from a table: a logarithm more per score, no loads (64 a row and tile) and no registers for them.
 //
+//   CAP: softmax over soft-capped scores, cap * tanh(scaled score / cap).
+//
 //   Pages past the entry's last page are read as the last page again (finite values the mask removes).
 //   Every mbarrier wait is bounded; one that runs out sets *status and all roles leave their loops.
 //
@@ -94,13 +96,14 @@ __device__ __forceinline__ uint32_t pt_pack(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <bool SIG, bool LOGB>
+template <bool SIG, bool LOGB, bool CAP>
 __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5_kernel(
     const __grid_constant__ CUtensorMap kv_map, const __nv_bfloat16* __restrict__ qkv, int row_stride,
     __nv_bfloat16* __restrict__ out, const int* __restrict__ block_table, int bt_stride, const int* __restrict__ entry_qstart,
-    const int* __restrict__ entry_kvlen, int first_entry, int n_entries, int nh, int nkv, float scale_log2, int window, int tpt,
+    const int* __restrict__ entry_kvlen, int first_entry, int n_entries, int nh, int nkv, float k_scale, int window, int tpt,
     int* __restrict__ status, const float* __restrict__ sink, const float* __restrict__ dist_bias, int dist_far, float inv_scale,
-    const float* __restrict__ log_bias) {
+    const float* __restrict__ log_bias, float cap_log2) {
+    const float scale_log2 = CAP ? 1.f : k_scale; // (capped scores are in base 2 already; k_scale is then the cap's factor)
     extern __shared__ __align__(1024) unsigned char smem[];
     if (t5_smem(smem) & 1023u) {                  // the swizzled tiles need 1 KB alignment; dynamic shared memory starts on it
         if (threadIdx.x == 0) atomicExch(status, 30);
@@ -321,6 +324,16 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
                         sv[c] = __float_as_uint(fmaf(db_row[max(0, min(rpos - kb - c, dist_far)) * nh], inv_scale, __uint_as_float(sv[c])));
                 }
             }
+            if constexpr (CAP) {                  // cap * tanh(score / cap) as 1 - 2 / (1 + 2^(k s)), one reciprocal for two scores
+#pragma unroll
+                for (int c = 0; c < PT_KEYS; c += 2) {
+                    const float a = 1.f + pt_ex2(fminf(__uint_as_float(sv[c]) * k_scale, 60.f));
+                    const float bb = 1.f + pt_ex2(fminf(__uint_as_float(sv[c + 1]) * k_scale, 60.f));
+                    const float rr = __fdividef(-2.f * cap_log2, a * bb);
+                    sv[c] = __float_as_uint(fmaf(rr, bb, cap_log2));
+                    sv[c + 1] = __float_as_uint(fmaf(rr, a, cap_log2));
+                }
+            }
             if (kb + PT_KEYS - 1 > rpos || kb < rlo) {        // the tile touches this row's causal or window edge
 #pragma unroll
                 for (int c = 0; c < PT_KEYS; ++c) {
@@ -453,10 +466,11 @@ IL_EXPORT int il_attn_prefill_tc5(const void* qkv, int row_stride, void* out, co
                                   int bt_stride, const int* entry_qstart, const int* entry_kvlen, int page_size, int first_entry,
                                   int n_entries, int n_tiles_total, int nh, int nkv, int hd, float scale, int window, int* status,
                                   const float* sink, const float* dist_bias, int dist_far, int sigmoid, const float* log_bias,
-                                  cudaStream_t stream) {
+                                  float cap, cudaStream_t stream) {
     if (n_tiles_total <= 0 || first_entry >= n_entries) return IL_OK;
     if (dist_bias && (dist_far < 0 || (long long)(dist_far + 1) * nh > 0x7fffffffLL)) return IL_BAD_ARG;
     if (log_bias && (!sigmoid || dist_bias)) return IL_BAD_ARG;
+    if (cap > 0.f && (sigmoid || dist_bias)) return IL_BAD_ARG;
     if (sigmoid && sink) return IL_BAD_ARG;       // a sink is a term of a softmax's denominator
     if (hd != HEAD_DIM || page_size != PT_PAGE || !kv_map || !status) return IL_UNSUPPORTED;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0) return IL_BAD_ARG;
@@ -468,7 +482,8 @@ IL_EXPORT int il_attn_prefill_tc5(const void* qkv, int row_stride, void* out, co
     static bool attr_set[64];
     if (dev >= 0 && dev < 64 && !attr_set[dev]) {
         cudaError_t e = cudaSuccess;
-        for (auto k : {attn_prefill_tc5_kernel<false, false>, attn_prefill_tc5_kernel<true, false>, attn_prefill_tc5_kernel<true, true>}) {
+        for (auto k : {attn_prefill_tc5_kernel<false, false, false>, attn_prefill_tc5_kernel<true, false, false>, attn_prefill_tc5_kernel<true, true, false>,
+                       attn_prefill_tc5_kernel<false, false, true>}) {
             if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, PT_SMEM);
             if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
         }
@@ -478,9 +493,11 @@ IL_EXPORT int il_attn_prefill_tc5(const void* qkv, int row_stride, void* out, co
     CUtensorMap map;
     memcpy(&map, kv_map, sizeof(map));
     dim3 grid(n_tiles_total, nkv);
-    (log_bias ? attn_prefill_tc5_kernel<true, true> : sigmoid ? attn_prefill_tc5_kernel<true, false> : attn_prefill_tc5_kernel<false, false>)<<<grid, PT_THREADS, PT_SMEM, stream>>>(
+    (log_bias ? attn_prefill_tc5_kernel<true, true, false> : sigmoid ? attn_prefill_tc5_kernel<true, false, false>
+              : cap > 0.f ? attn_prefill_tc5_kernel<false, false, true> : attn_prefill_tc5_kernel<false, false, false>)<<<grid, PT_THREADS, PT_SMEM, stream>>>(
         map, (const __nv_bfloat16*)qkv, row_stride, (__nv_bfloat16*)out, block_table, bt_stride, entry_qstart, entry_kvlen,
-        first_entry, n_entries, nh, nkv, scale * 1.4426950408889634f, window, PT_ROWS / G, status, sink, dist_bias, dist_far, 1.f / scale, log_bias);
+        first_entry, n_entries, nh, nkv, (cap > 0.f ? 2.f * scale / cap : scale) * 1.4426950408889634f, window, PT_ROWS / G, status, sink, dist_bias, dist_far, 1.f / scale, log_bias,
+        cap * 1.4426950408889634f);
     IL_LAUNCH_CHECK();
     return IL_OK;
 }

@@ -105,7 +105,13 @@ __device__ __forceinline__ float il_clamped_glu(float g, float u, float limit, f
 }
 // The gate of a gated feed-forward by number: 1 SiLU, 2 the tanh form of GELU, 3 the clamped gate (which has two numbers
 // of its own, limit and alpha).
-enum { IL_ACT_SILU = 1, IL_ACT_GELU_TANH = 2, IL_ACT_CLAMPED = 3 };
+// Activations of a product that stand on their own: 4 the square of relu; 5 the tanh form of GELU times a row of a table that
+// the row's token names.
+enum { IL_ACT_SILU = 1, IL_ACT_GELU_TANH = 2, IL_ACT_CLAMPED = 3, IL_ACT_RELU2 = 4, IL_ACT_GELU_TANH_ROW = 5 };
+__device__ __forceinline__ float il_relu2(float z) {
+    z = fmaxf(z, 0.f);
+    return __fmul_rn(z, z);
+}
 
 // 1 / (1 + 2^-v), the logistic function of v / log2(e): -inf gives 0. Exponential and reciprocal by the fast units (relative
 // error near 2^-21).
@@ -113,6 +119,14 @@ __device__ __forceinline__ float il_sigmoid_log2_fast(float v) {
     float e;
     asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(-v));
     return __fdividef(1.f, 1.f + fminf(e, 1e38f));
+}
+
+// A capped score in the exponent's base: c * tanh(x) where 2^(k s) = e^(2x), so k = 2 log2(e) scale / cap and c = cap log2(e).
+// tanh(x) = 1 - 2 / (1 + e^(2x)); exponential and reciprocal by the fast units (absolute error near 2^-21 c).
+__device__ __forceinline__ float il_cap_log2_fast(float s, float k, float c) {
+    float e;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(s * k));
+    return fmaf(-2.f * c, __fdividef(1.f, 1.f + fminf(e, 1e38f)), c);
 }
 
 // ---- programmatic dependent launch --------------------------------------------------------------

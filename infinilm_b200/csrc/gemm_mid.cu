@@ -84,7 +84,7 @@ enum { GM_PLAIN = 0, GM_GLU = 1 };
 struct GmParams {
     int M, N, K;                                  // N: output columns (SwiGLU: the intermediate size; W has 2N rows)
     int mode, n_acc;                              // accumulators per unit: 1 plain, 2 SwiGLU (gate, up)
-    int act;                                      // the gate of the SwiGLU form: IL_ACT_SILU, IL_ACT_GELU_TANH or IL_ACT_CLAMPED
+    int act;                                      // the gate of the SwiGLU form: IL_ACT_SILU, IL_ACT_GELU_TANH or IL_ACT_CLAMPED; plain: 0 or IL_ACT_RELU2
     float act_limit, act_alpha;                   // the clamped gate's two numbers
     int NB, n_bb;                                 // activation rows per unit (a multiple of 16), blocks of them
     int n_issuers;                                // threads that issue products, each into an accumulator of its own
@@ -302,6 +302,10 @@ __global__ void __launch_bounds__(GM_THREADS, 1) gemm_mid_kernel(const __grid_co
                     }
 #pragma unroll
                     for (int j = 0; j < 16; ++j) y[j] = __fmaf_rn(p.alpha, sum[j], bg);
+                    if (p.act == IL_ACT_RELU2) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) y[j] = il_relu2(y[j]);
+                    }
                 }
                 if (n_ok) {
                     if (p.out_kind == IL_F32) {
@@ -399,21 +403,23 @@ static int gm_pick_nb(int Mp, int n_tiles, int n_sm) {
 
 IL_EXPORT int il_gemm_mid_max_rows() { return GM_MAX_ROWS; }
 
-// glu = 1: W is [2N, K] (N gate rows, then N up rows), bias [2N], out[M,N] = silu(alpha*x.Wg^T + bg) * (alpha*x.Wu^T + bu); glu = 2: gelu_tanh for silu; glu = 3: the clamped gate.
+// glu = 1: W is [2N, K] (N gate rows, then N up rows), bias [2N], out[M,N] = silu(alpha*x.Wg^T + bg) * (alpha*x.Wu^T + bu); glu = 2: gelu_tanh for silu; glu = 3: the clamped gate;
+// glu = 4: W is [N, K], out[M,N] = relu(alpha*x.W^T + b)^2 (bfloat16).
 // nb: activation rows per unit, bm_want: weight rows per tile, 64 or 128 (0: chosen here).
 IL_EXPORT int il_gemm_mid(const void* x, int ldx, const void* W, int ldw, void* out, int out_kind, int ldo, const float* bias,
-                          float alpha, int M, int N, int K, int glu, int nb, int bm_want, float act_limit, float act_alpha, int* status,
+                          float alpha, int M, int N, int K, int act, int nb, int bm_want, float act_limit, float act_alpha, int* status,
                           cudaStream_t stream) {
     if (M <= 0 || N <= 0) return IL_OK;
     if (M > GM_MAX_ROWS || K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || ldx < K || ldw < K || ldo < N || !status) return IL_UNSUPPORTED;
     if (((uintptr_t)x & 15) || ((uintptr_t)W & 15)) return IL_UNSUPPORTED;
     if (out_kind != IL_F32 && out_kind != IL_BF16) return IL_BAD_ARG;
-    if (glu && out_kind != IL_BF16) return IL_UNSUPPORTED;
+    if (act && out_kind != IL_BF16) return IL_UNSUPPORTED;
+    const int glu = act == IL_ACT_RELU2 ? 0 : act;
     const int n_sm = gm_sm_count();
     const int Mp = (M + 15) & ~15;
 
     GmParams p;
-    p.M = M; p.N = N; p.K = K; p.mode = glu ? GM_GLU : GM_PLAIN; p.n_acc = glu ? 2 : 1; p.act = glu == 3 ? IL_ACT_CLAMPED : glu == 2 ? IL_ACT_GELU_TANH : IL_ACT_SILU;
+    p.M = M; p.N = N; p.K = K; p.mode = glu ? GM_GLU : GM_PLAIN; p.n_acc = glu ? 2 : 1; p.act = act == IL_ACT_RELU2 || act == 0 ? act : act == 3 ? IL_ACT_CLAMPED : act == 2 ? IL_ACT_GELU_TANH : IL_ACT_SILU;
     p.act_limit = act_limit; p.act_alpha = act_alpha;
     // tiles of 128 rows where that still gives (nearly) every SM a unit at whole activation blocks: a product of M = 64
     // covers 2 KB of weights and the tensor pipe takes some 80 clocks for it, which holds an SM to about 50 GB/s

@@ -64,15 +64,25 @@ __device__ __forceinline__ void gs_norm_finish(float* rstd_s, const float (&pv)[
     }
 }
 
-// NT: 8-row groups of x (1: M <= 8, 2: M <= 16). GLU: 0 plain, 1 SwiGLU, 2 the same with the tanh form of GELU as the gate, 3 with the clamped gate (act_limit, act_alpha) (W holds N gate rows, then N up rows). U: blocks in flight.
+// What the epilogue of ACT_GELU_TANH_ROW multiplies by: row ids[m] of a table (bfloat16), columns off .. off + dim; columns of the
+// product from dim on give 0.
+struct GsRowMul {
+    const int* ids;
+    const __nv_bfloat16* table;
+    int ld, off, dim, vocab;
+};
+__host__ __device__ constexpr bool gs_gated(int glu) { return glu >= IL_ACT_SILU && glu <= IL_ACT_CLAMPED; }
+
+// NT: 8-row groups of x (1: M <= 8, 2: M <= 16). GLU: 0 plain, 4 plain with relu(.)^2, 5 plain with gelu_tanh(.) * a table's row; 1 SwiGLU, 2 the same with the tanh form of GELU as the gate, 3 with the clamped gate (act_limit, act_alpha) (W holds N gate rows, then N up rows). U: blocks in flight.
 // NRM: the activations may come without their norm's 1/rms (`ni`); the SwiGLU form always can, the plain form as a variant of its own.
-template <int NT, int GLU, int U, typename TO, bool NRM = (GLU != 0)>
+template <int NT, int GLU, int U, typename TO, bool NRM = gs_gated(GLU)>
 __global__ void __launch_bounds__(GS_WARPS * 32, 2) gemm_skinny_kernel(const __nv_bfloat16* __restrict__ x, int ldx,
                                                                     const __nv_bfloat16* __restrict__ W, int ldw, TO* __restrict__ out,
                                                                     int ldo, const float* __restrict__ bias, float alpha, int M, int N, int K,
-                                                                    const GsNormIn ni, float act_limit, float act_alpha) {
+                                                                    const GsNormIn ni, float act_limit, float act_alpha, const GsRowMul rm) {
     constexpr int NW = 1;
-    constexpr int ROWS = GLU ? 8 : 16;            // outputs per activation row and tile: 16 rows, or 8 gate rows with their 8 up rows
+    constexpr bool GATED = gs_gated(GLU);
+    constexpr int ROWS = GATED ? 8 : 16;           // outputs per activation row and tile: 16 rows, or 8 gate rows with their 8 up rows
     __shared__ float part[GS_WARPS][NW][NT][16][8];
     __shared__ float rstd_s[NT * 8];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -83,9 +93,9 @@ __global__ void __launch_bounds__(GS_WARPS * 32, 2) gemm_skinny_kernel(const __n
     for (int s = 0; s < NW; ++s)
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-            int n = GLU ? n0 + r : n0 + r + 8 * h;
+            int n = GATED ? n0 + r : n0 + r + 8 * h;
             if (n > N - 1) n = N - 1;             // rows past the end are computed and dropped
-            wrow[s][h] = W + ((size_t)(GLU ? h : 0) * N + n) * ldw;
+            wrow[s][h] = W + ((size_t)(GATED ? h : 0) * N + n) * ldw;
         }
     il_pdl_begin();
     float pv[NT][8];
@@ -149,11 +159,16 @@ __global__ void __launch_bounds__(GS_WARPS * 32, 2) gemm_skinny_kernel(const __n
 #pragma unroll
         for (int w = 0; w < GS_WARPS; ++w) {
             s0 += part[w][0][t][nl][mc];
-            if (GLU) s1 += part[w][0][t][nl + 8][mc];
+            if (GATED) s1 += part[w][0][t][nl + 8][mc];
         }
         const float an = NRM ? __fmul_rn(alpha, rstd_s[m]) : alpha;     // the norm's 1/rms, where the activations came without it
         float y = __fmaf_rn(an, s0, bias ? bias[n] : 0.f);      // spelled out as one fused multiply-add: the same bits from every build of this line
-        if (GLU) {
+        if (GLU == IL_ACT_RELU2) y = il_relu2(y);
+        if (GLU == IL_ACT_GELU_TANH_ROW) {
+            const int id = rm.ids[m];
+            y = (n < rm.dim && id >= 0 && id < rm.vocab) ? il_gelu_tanh_mul_fast(y, __bfloat162float(rm.table[(size_t)id * rm.ld + rm.off + n])) : 0.f;
+        }
+        if (GATED) {
             const float u = __fmaf_rn(an, s1, bias ? bias[N + n] : 0.f);
             y = GLU == 3 ? il_clamped_glu_fast(y, u, act_limit, act_alpha) : GLU == 2 ? il_gelu_tanh_mul_fast(y, u) : il_silu_mul_fast(y, u);
         }
@@ -161,18 +176,19 @@ __global__ void __launch_bounds__(GS_WARPS * 32, 2) gemm_skinny_kernel(const __n
     }
 }
 
-template <int NT, int GLU, typename TO, bool NRM = (GLU != 0)>
+template <int NT, int GLU, typename TO, bool NRM = gs_gated(GLU)>
 static cudaError_t gs_launch(const void* x, int ldx, const void* W, int ldw, void* out, int ldo, const float* bias, float alpha, int M, int N,
                       int K, cudaStream_t stream, const GsNormIn& ni = GsNormIn{nullptr, 0, 0.f, 0.f}, float act_limit = 0.f,
-                      float act_alpha = 0.f) {
+                      float act_alpha = 0.f, const GsRowMul& rm = GsRowMul{nullptr, nullptr, 0, 0, 0, 0}) {
     constexpr int U = NT == 1 ? 8 : 4;
-    constexpr int ROWS = GLU ? 8 : 16;
+    constexpr int ROWS = gs_gated(GLU) ? 8 : 16;
     return il_launch(gemm_skinny_kernel<NT, GLU, U, TO, NRM>, dim3((N + ROWS - 1) / ROWS), dim3(GS_WARPS * 32), 0, stream,
-              (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)out, ldo, bias, alpha, M, N, K, ni, act_limit, act_alpha);
+              (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, ldw, (TO*)out, ldo, bias, alpha, M, N, K, ni, act_limit, act_alpha, rm);
 }
 
 // glu = 1: W is [2N, K] (N gate rows, then N up rows), bias [2N], out[M,N] = silu(alpha*x.Wg^T + bg) * (alpha*x.Wu^T + bu);
-// glu = 2: the same with gelu_tanh in place of silu; glu = 3: the clamped gate with its two numbers.
+// glu = 2: the same with gelu_tanh in place of silu; glu = 3: the clamped gate with its two numbers; glu = 4: W is [N, K] and
+// out[M,N] = relu(alpha*x.W^T + b)^2. (These write bfloat16.)
 // norm_partial (may be null): x is residual * norm weight and still wants its 1/rms, from these sums of squares
 // [M][n_partial] (n_partial <= 256, H = the width they were summed over).
 IL_EXPORT int il_gemm_skinny(const void* x, int ldx, const void* W, int ldw, void* out, int out_kind, int ldo, const float* bias,
@@ -186,7 +202,9 @@ IL_EXPORT int il_gemm_skinny(const void* x, int ldx, const void* W, int ldw, voi
     if (glu && out_kind != IL_BF16) return IL_UNSUPPORTED;
     cudaError_t e;
     if (M <= 8) {
-        if (glu == 3) e = gs_launch<1, 3, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni, act_limit, act_alpha);
+        if (glu == 4 && norm_partial) e = gs_launch<1, 4, __nv_bfloat16, true>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
+        else if (glu == 4) e = gs_launch<1, 4, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream);
+        else if (glu == 3) e = gs_launch<1, 3, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni, act_limit, act_alpha);
         else if (glu == 2) e = gs_launch<1, 2, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (glu) e = gs_launch<1, 1, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (norm_partial && out_kind == IL_BF16) e = gs_launch<1, 0, __nv_bfloat16, true>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
@@ -194,7 +212,9 @@ IL_EXPORT int il_gemm_skinny(const void* x, int ldx, const void* W, int ldw, voi
         else if (out_kind == IL_BF16) e = gs_launch<1, 0, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream);
         else e = gs_launch<1, 0, float>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream);
     } else {
-        if (glu == 3) e = gs_launch<2, 3, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni, act_limit, act_alpha);
+        if (glu == 4 && norm_partial) e = gs_launch<2, 4, __nv_bfloat16, true>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
+        else if (glu == 4) e = gs_launch<2, 4, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream);
+        else if (glu == 3) e = gs_launch<2, 3, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni, act_limit, act_alpha);
         else if (glu == 2) e = gs_launch<2, 2, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (glu) e = gs_launch<2, 1, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
         else if (norm_partial && out_kind == IL_BF16) e = gs_launch<2, 0, __nv_bfloat16, true>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream, ni);
@@ -202,6 +222,21 @@ IL_EXPORT int il_gemm_skinny(const void* x, int ldx, const void* W, int ldw, voi
         else if (out_kind == IL_BF16) e = gs_launch<2, 0, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream);
         else e = gs_launch<2, 0, float>(x, ldx, W, ldw, out, ldo, bias, alpha, M, N, K, stream);
     }
+    if (e != cudaSuccess) return 1000 + (int)e;
+    IL_LAUNCH_CHECK();
+    return IL_OK;
+}
+
+// out[m, n] = gelu_tanh(x . W^T) * table[ids[m], off + n] (bfloat16; columns n >= dim give 0): the gate of a token's own table row.
+IL_EXPORT int il_gemm_skinny_gelu_row(const void* x, int ldx, const void* W, int ldw, void* out, int ldo, int M, int N, int K, const int* ids,
+                                      const void* table, int ldt, int off, int dim, int vocab, cudaStream_t stream) {
+    if (M <= 0 || N <= 0) return IL_OK;
+    if (M > 16 || K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || ldx < K || ldw < K || ldo < N) return IL_UNSUPPORTED;
+    if (!ids || !table || dim <= 0 || dim > N || off < 0 || off + dim > ldt || vocab <= 0) return IL_BAD_ARG;
+    const GsNormIn ni{nullptr, 0, 0.f, 0.f};
+    const GsRowMul rm{ids, (const __nv_bfloat16*)table, ldt, off, dim, vocab};
+    const cudaError_t e = M <= 8 ? gs_launch<1, 5, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, nullptr, 1.f, M, N, K, stream, ni, 0.f, 0.f, rm)
+                                 : gs_launch<2, 5, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, nullptr, 1.f, M, N, K, stream, ni, 0.f, 0.f, rm);
     if (e != cudaSuccess) return 1000 + (int)e;
     IL_LAUNCH_CHECK();
     return IL_OK;

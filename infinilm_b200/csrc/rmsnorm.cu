@@ -336,6 +336,158 @@ IL_EXPORT int il_norm_add_norm(float* resid, const void* branch, const int* pos,
     return IL_OK;
 }
 
+// ---- several branches joined in one pass ----------------------------------------------------------------------------------
+//   total    = sum_i scale_i * cs_i * (y_i, or y_i / sqrt(mean(y_i^2) + eps_i) * nw_i)       up to BS_MAX_TERMS branches y_i [rows, H]
+//   resid[r] += total (resid null: not)                                                       f32
+//   copy[r]   = resid[r], or total where resid is null, in the activations' type (null: not)
+//   out[r]    = resid[r] / sqrt(mean(resid[r]^2) + eps_n) * wn (null: not)
+// nw_i (the branch's own norm) and cs_i (a factor per column) are each optional. What stands behind the sublayers of a block that
+// run side by side on one input. One block per row with a fixed thread count; a thread's columns stay in registers, the
+// branches are added in their order.
+#define BS_MAX_TERMS 4
+struct BsTerm {
+    const void* y;
+    const void* nw;
+    const void* cs;
+    int nw_kind, cs_kind;
+    float scale, eps;
+};
+struct BsTerms { BsTerm t[BS_MAX_TERMS]; };
+
+template <typename TA, int VW, int MAXV, int NT>
+__global__ void __launch_bounds__(256) branch_sum_kernel(float* resid, const BsTerms ts, TA* copy, const void* __restrict__ wn, int wn_kind,
+                                                         float eps_n, TA* __restrict__ out, int H) {
+    __shared__ float red[NT + 1][8];
+    const int r = blockIdx.x, nv = (H + VW - 1) / VW, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    il_pdl_wait();
+    float4 c[NT][MAXV], x[MAXV];
+    float* rr = resid ? resid + (size_t)r * H : nullptr;
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int k = 0; k < MAXV; ++k) {
+            const int v = threadIdx.x + k * 256;
+            c[i][k] = v < nv ? NanVec<TA, VW>::ld((const TA*)ts.t[i].y + (size_t)r * H + v * VW) : zero;
+        }
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+        const int v = threadIdx.x + k * 256;
+        x[k] = (rr && v < nv) ? NanVec<float, VW>::ld(rr + v * VW) : zero;
+    }
+    bool any = false;
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+        if (!ts.t[i].nw) continue;                // (the same for the whole grid)
+        any = true;
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < MAXV; ++k) ss += c[i][k].x * c[i][k].x + c[i][k].y * c[i][k].y + c[i][k].z * c[i][k].z + c[i][k].w * c[i][k].w;
+        ss = il_warp_sum(ss);
+        if (lane == 0) red[i][warp] = ss;
+    }
+    if (any) __syncthreads();
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+        const BsTerm& t = ts.t[i];
+        float f = t.scale;
+        if (t.nw) {
+            float ss = 0.f;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) ss += red[i][w];
+            f *= 1.f / sqrtf(ss / (float)H + t.eps);
+        }
+#pragma unroll
+        for (int k = 0; k < MAXV; ++k) {
+            const int v = threadIdx.x + k * 256;
+            if (v >= nv) continue;
+            float4 w = make_float4(f, f, f, f);
+            if (t.nw) {
+                const float4 a = nan_w<VW>(t.nw, t.nw_kind, v * VW);
+                w.x *= a.x, w.y *= a.y, w.z *= a.z, w.w *= a.w;
+            }
+            if (t.cs) {
+                const float4 a = nan_w<VW>(t.cs, t.cs_kind, v * VW);
+                w.x *= a.x, w.y *= a.y, w.z *= a.z, w.w *= a.w;
+            }
+            x[k].x = fmaf(w.x, c[i][k].x, x[k].x), x[k].y = fmaf(w.y, c[i][k].y, x[k].y);
+            x[k].z = fmaf(w.z, c[i][k].z, x[k].z), x[k].w = fmaf(w.w, c[i][k].w, x[k].w);
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+        const int v = threadIdx.x + k * 256;
+        if (v >= nv) continue;
+        if (rr) NanVec<float, VW>::st(rr + v * VW, x[k]);
+        if (copy) NanVec<TA, VW>::st(copy + (size_t)r * H + v * VW, x[k]);
+    }
+    if (!out) return;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) ss += x[k].x * x[k].x + x[k].y * x[k].y + x[k].z * x[k].z + x[k].w * x[k].w;
+    ss = il_warp_sum(ss);
+    if (lane == 0) red[NT][warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) ss += red[NT][w];
+    const float kn = 1.f / sqrtf(ss / (float)H + eps_n);
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+        const int v = threadIdx.x + k * 256;
+        if (v >= nv) continue;
+        const float4 b = nan_w<VW>(wn, wn_kind, v * VW);
+        NanVec<TA, VW>::st(out + (size_t)r * H + v * VW, make_float4(x[k].x * kn * b.x, x[k].y * kn * b.y, x[k].z * kn * b.z, x[k].w * kn * b.w));
+    }
+}
+
+template <typename TA, int NT>
+static int bs_launch(float* resid, const BsTerms& ts, void* copy, const void* wn, int wn_kind, float eps_n, void* out, int n_rows, int H,
+                     cudaStream_t stream) {
+    uintptr_t all = (uintptr_t)resid | (uintptr_t)copy | (uintptr_t)wn | (uintptr_t)out;
+    for (int i = 0; i < NT; ++i) all |= (uintptr_t)ts.t[i].y | (uintptr_t)ts.t[i].nw | (uintptr_t)ts.t[i].cs;
+    const bool vec = (H & 3) == 0 && (all & 15) == 0;
+#define BS_GO(VW, MAXV) \
+    IL_LAUNCH((branch_sum_kernel<TA, VW, MAXV, NT>), n_rows, 256, 0, stream, resid, ts, (TA*)copy, wn, wn_kind, eps_n, (TA*)out, H)
+    if (vec && H <= 256 * 4) BS_GO(4, 1);
+    else if (vec && H <= 256 * 4 * 2) BS_GO(4, 2);
+    else if (vec && H <= 256 * 4 * 4) BS_GO(4, 4);
+    else if (vec && H <= 256 * 4 * 8) BS_GO(4, 8);
+    else if (H <= 256 * 4) BS_GO(1, 4);
+    else if (H <= 256 * 16) BS_GO(1, 16);
+    else return IL_UNSUPPORTED;
+#undef BS_GO
+    return IL_OK;
+}
+
+// The branches come as parallel arrays of n_terms entries on the host.
+IL_EXPORT int il_branch_sum(float* resid, const void* const* y, const void* const* nw, const int* nw_kind, const void* const* cs, const int* cs_kind,
+                            const float* scale, const float* eps, int n_terms, void* copy, const void* wn, int wn_kind, float eps_n, void* out,
+                            int act_kind, int n_rows, int H, cudaStream_t stream) {
+    if (n_rows <= 0) return IL_OK;
+    if (n_terms <= 0 || n_terms > BS_MAX_TERMS || H <= 0 || (!resid && !copy) || (out && (!wn || !resid))) return IL_BAD_ARG;
+    if (act_kind != IL_F32 && act_kind != IL_BF16) return IL_BAD_ARG;
+    BsTerms ts = {};
+    for (int i = 0; i < n_terms; ++i) {
+        if (!y[i]) return IL_BAD_ARG;
+        ts.t[i] = BsTerm{y[i], nw[i], cs[i], nw_kind[i], cs_kind[i], scale[i], eps[i]};
+    }
+    int rc = IL_OK;
+#define BS_PICK(TA)                                                                                           \
+    do {                                                                                                      \
+        if (n_terms == 1) rc = bs_launch<TA, 1>(resid, ts, copy, wn, wn_kind, eps_n, out, n_rows, H, stream); \
+        else if (n_terms == 2) rc = bs_launch<TA, 2>(resid, ts, copy, wn, wn_kind, eps_n, out, n_rows, H, stream); \
+        else if (n_terms == 3) rc = bs_launch<TA, 3>(resid, ts, copy, wn, wn_kind, eps_n, out, n_rows, H, stream); \
+        else rc = bs_launch<TA, 4>(resid, ts, copy, wn, wn_kind, eps_n, out, n_rows, H, stream);              \
+    } while (0)
+    if (act_kind == IL_F32) BS_PICK(float);
+    else BS_PICK(__nv_bfloat16);
+#undef BS_PICK
+    if (rc != IL_OK) return rc;
+    IL_LAUNCH_CHECK();
+    return IL_OK;
+}
+
 // rows of f32 copied into the activations' type (the first sublayer's input, where no norm_add ran before it)
 template <typename TA>
 __global__ void cast_rows_kernel(const float* x, TA* out, size_t total) {

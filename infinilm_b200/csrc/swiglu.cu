@@ -52,6 +52,43 @@ __global__ void swiglu_vec_kernel(const TA* __restrict__ gu, TA* __restrict__ ou
     }
 }
 
+// ---- activations that stand on their own ---------------------------------------------------------------------------------
+// y[i] = relu(z[i])^2, VEC neighbours a thread (out may be z).
+template <typename TA, int VEC>
+__global__ void relu2_kernel(const TA* z, TA* out, size_t total_vec) {
+    il_pdl_wait();
+    const size_t stride = (size_t)gridDim.x * blockDim.x;
+    for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total_vec; idx += stride) {
+        if (VEC == 1) {
+            out[idx] = il_from_f<TA>(il_relu2(il_to_f(z[idx])));
+        } else {
+            uint4 q = reinterpret_cast<const uint4*>(z)[idx];
+            TA* p = reinterpret_cast<TA*>(&q);
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) p[k] = il_from_f<TA>(il_relu2(il_to_f(p[k])));
+            reinterpret_cast<uint4*>(out)[idx] = q;
+        }
+    }
+}
+
+// out[t, n] = gelu_tanh(z[t, n]) * table[ids[t], off + n] for n < dim, 0 for dim <= n < ldo: a token's own row of a table, gated.
+template <typename TA>
+__global__ void gelu_row_kernel(const TA* z, int ldz, const int* __restrict__ ids, const TA* __restrict__ table, int ldt, int off, int dim, int vocab,
+                                TA* __restrict__ out, int ldo, long long total) {
+    il_pdl_wait();
+    const long long stride = (long long)gridDim.x * blockDim.x;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
+        const long long t = i / ldo;
+        const int n = (int)(i - t * ldo), id = ids[t];
+        float y = 0.f;
+        if (n < dim && id >= 0 && id < vocab) {   // (the host rejects other ids before launch; never read out of range)
+            const float g = il_to_f(z[t * ldz + n]), e = il_to_f(table[(size_t)id * ldt + off + n]);
+            y = sizeof(TA) == 2 ? il_gelu_tanh_mul_fast(g, e) : il_gelu_tanh_mul(g, e);
+        }
+        out[i] = il_from_f<TA>(y);
+    }
+}
+
 template <typename TA>
 __global__ void add_bias_kernel(TA* __restrict__ y, const void* __restrict__ b, int b_kind, int N, size_t total) {
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -110,6 +147,41 @@ IL_EXPORT int il_add_bias(void* y, int act_kind, const void* bias, int bias_kind
         add_bias_kernel<float><<<grid, threads, 0, stream>>>((float*)y, bias, bias_kind, N, total);
     else if (act_kind == IL_BF16)
         add_bias_kernel<__nv_bfloat16><<<grid, threads, 0, stream>>>((__nv_bfloat16*)y, bias, bias_kind, N, total);
+    else
+        return IL_BAD_ARG;
+    IL_LAUNCH_CHECK();
+    return IL_OK;
+}
+
+IL_EXPORT int il_relu2(const void* z, void* out, int act_kind, long long total, cudaStream_t stream) {
+    if (total <= 0) return IL_OK;
+    if (act_kind != IL_F32 && act_kind != IL_BF16) return IL_BAD_ARG;
+    const int vec = act_kind == IL_F32 ? 4 : 8;
+    const bool v = total % vec == 0 && (((uintptr_t)z | (uintptr_t)out) & 15) == 0;
+    const long long n = v ? total / vec : total, g = (n + 255) / 256;
+    const int blocks = (int)(g > 148 * 32 ? 148 * 32 : g);
+    if (act_kind == IL_F32) {
+        if (v) IL_LAUNCH((relu2_kernel<float, 4>), blocks, 256, 0, stream, (const float*)z, (float*)out, (size_t)n);
+        else IL_LAUNCH((relu2_kernel<float, 1>), blocks, 256, 0, stream, (const float*)z, (float*)out, (size_t)n);
+    } else {
+        if (v) IL_LAUNCH((relu2_kernel<__nv_bfloat16, 8>), blocks, 256, 0, stream, (const __nv_bfloat16*)z, (__nv_bfloat16*)out, (size_t)n);
+        else IL_LAUNCH((relu2_kernel<__nv_bfloat16, 1>), blocks, 256, 0, stream, (const __nv_bfloat16*)z, (__nv_bfloat16*)out, (size_t)n);
+    }
+    IL_LAUNCH_CHECK();
+    return IL_OK;
+}
+
+IL_EXPORT int il_gelu_row(const void* z, int act_kind, int ldz, const int* ids, const void* table, int ldt, int off, int dim, int vocab, void* out,
+                          int ldo, int T, cudaStream_t stream) {
+    if (T <= 0) return IL_OK;
+    if (dim <= 0 || ldz < dim || ldo < dim || off < 0 || off + dim > ldt || vocab <= 0) return IL_BAD_ARG;
+    const long long total = (long long)T * ldo, g = (total + 255) / 256;
+    const int blocks = (int)(g > 148 * 16 ? 148 * 16 : g);
+    if (act_kind == IL_F32)
+        IL_LAUNCH(gelu_row_kernel<float>, blocks, 256, 0, stream, (const float*)z, ldz, ids, (const float*)table, ldt, off, dim, vocab, (float*)out, ldo, total);
+    else if (act_kind == IL_BF16)
+        IL_LAUNCH(gelu_row_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (const __nv_bfloat16*)z, ldz, ids, (const __nv_bfloat16*)table, ldt, off, dim, vocab,
+                  (__nv_bfloat16*)out, ldo, total);
     else
         return IL_BAD_ARG;
     IL_LAUNCH_CHECK();

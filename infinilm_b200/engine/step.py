@@ -103,6 +103,7 @@ class StepContext:
     max_qlen: int = 0
     max_kvlen: int = 0
     tap: Optional[Callable] = None                # debug hook: tap(name, resid, pending)
+    shared: dict = field(default_factory=dict)    # device rows a layer leaves for later layers of the same step, by name
     lengths_are_bounds: bool = False              # h_qlen / h_kvlen are upper bounds (a step replayed as a graph)
 
     def prompt_tiles(self, tokens_per_tile: int) -> int:

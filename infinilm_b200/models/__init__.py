@@ -5,7 +5,7 @@ import importlib
 
 from .causal_lm import CausalLM
 
-BUILTIN = ("minicpm4", "nirozen", "gopitar", "somipel", "zokuzen", "zibinex")
+BUILTIN = ("minicpm4", "nirozen", "gopitar", "somipel", "zokuzen", "zibinex", "gukosun")
 
 
 def register_builtin() -> None:

@@ -23,8 +23,8 @@ class CausalLM:
         self.blocks = []
         for ls in spec.layers:
             arr = part_class("arrangement", ls.arrangement)
-            if (ls.ffn is None) != (ls.ffn_norm is None):
-                raise ValueError("a layer has a feed-forward and its norm, or neither")
+            if ls.ffn_norm is not None if arr.one_norm else (ls.ffn is None) != (ls.ffn_norm is None):
+                raise ValueError("a layer has a feed-forward and its norm, or neither (or its sublayers share one norm)")
             self.blocks.append(arr(build_part("norm", ls.mixer_norm, dtype), build_part("mixer", ls.mixer, dtype),
                                    None if ls.ffn_norm is None else build_part("norm", ls.ffn_norm, dtype),
                                    None if ls.ffn is None else build_part("feed_forward", ls.ffn, dtype), ls.params))
@@ -32,6 +32,10 @@ class CausalLM:
         self.head = build_part("head", spec.head, dtype)
         self.order = list(spec.order)
         self.pass_vectors = None if spec.pass_vectors is None else build_part("embedding", spec.pass_vectors, dtype)
+        self.token_table = None if spec.token_table is None else build_part("embedding", spec.token_table, dtype)
+        for b in self.blocks:
+            if b.takes_token_table:
+                b.set_token_table(self.token_table)
         for i, st in enumerate(self.order):
             if st.add_row is not None:
                 if self.pass_vectors is None or not 0 <= st.add_row < self.pass_vectors.rows:
@@ -57,6 +61,8 @@ class CausalLM:
             out.extend(b.parts())
         if self.pass_vectors is not None:
             out.append(self.pass_vectors)
+        if self.token_table is not None:
+            out.append(self.token_table)
         out += [self.final_norm, self.head]
         return out
 

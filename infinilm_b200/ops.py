@@ -154,6 +154,7 @@ def add_rmsnorm(resid: torch.Tensor, branch: Optional[torch.Tensor], branch_scal
 
 
 ACT_SILU, ACT_GELU_TANH, ACT_CLAMPED = 1, 2, 3    # the gate of a gated feed-forward
+ACT_RELU2 = 4                                     # an activation without a gate: relu(z)^2
 
 
 def _act_args(act: int, act_params):
@@ -179,6 +180,53 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, act: int = ACT_SILU, act_pa
     f = _fn("swiglu", "il_swiglu", [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p, _c_void_p])
     limit, alpha = _act_args(act, act_params)
     _check(f(_ptr(gate_up), _ptr(out), kind_of(out.dtype), T, I2 // 2, int(act), limit, alpha, _ptr(row_scale), _stream()), "swiglu")
+
+
+def relu2(z: torch.Tensor, out: torch.Tensor) -> None:
+    """out = relu(z)^2; contiguous tensors of one shape and dtype (out may be z)."""
+    _need_cuda(z, out)
+    if z.shape != out.shape or z.dtype != out.dtype:
+        raise KernelError("relu2: one shape and dtype")
+    _contig("z", z), _contig("out", out)
+    f = _fn("swiglu", "il_relu2", [_c_void_p, _c_void_p, _c_int, ctypes.c_longlong, _c_void_p])
+    _check(f(_ptr(z), _ptr(out), kind_of(z.dtype), z.numel(), _stream()), "relu2")
+
+
+def _check_row_table(name: str, ids: torch.Tensor, table: torch.Tensor, off: int, dim: int, T: int, dtype) -> None:
+    if ids.dtype != torch.int32 or ids.numel() < T or not ids.is_contiguous():
+        raise KernelError(f"{name}: ids int32 [T]")
+    if table.dtype != dtype or table.dim() != 2 or table.stride(1) != 1 or off < 0 or dim <= 0 or off + dim > table.shape[1]:
+        raise KernelError(f"{name}: table [vocab, >= off + dim] of the activations' dtype")
+
+
+def gelu_row(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, off: int, dim: int, out: torch.Tensor) -> None:
+    """out[t, n] = gelu_tanh(z[t, n]) * table[ids[t], off + n] for n < dim, 0 in out's columns behind them."""
+    _need_cuda(z, ids, table, out)
+    T = z.shape[0]
+    _check_row_table("gelu_row", ids, table, off, dim, T, z.dtype)
+    if z.stride(1) != 1 or z.shape[1] < dim or out.dtype != z.dtype or out.shape[0] != T or out.shape[1] < dim or not out.is_contiguous():
+        raise KernelError("gelu_row: z [T, >= dim], out [T, >= dim] contiguous, one dtype")
+    f = _fn("swiglu", "il_gelu_row", [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int,
+                                      _c_void_p])
+    _check(f(_ptr(z), kind_of(z.dtype), z.stride(0), _ptr(ids), _ptr(table), table.stride(0), off, dim, table.shape[0], _ptr(out), out.shape[1], T,
+             _stream()), "gelu_row")
+
+
+def gemm_skinny_gelu_row(x: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, off: int, dim: int, out: torch.Tensor) -> None:
+    """out[m, n] = gelu_tanh(x @ w^T)[m, n] * table[ids[m], off + n] for n < dim (0 behind them): up to 16 bfloat16 rows, the
+    weight-streaming product with that in its epilogue."""
+    _need_cuda(x, w, ids, table, out)
+    M, K = x.shape
+    N = w.shape[0]
+    _check_row_table("gemm_skinny_gelu_row", ids, table, off, dim, M, torch.bfloat16)
+    if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != K or tuple(out.shape) != (M, N) or out.dtype != torch.bfloat16 or dim > N:
+        raise KernelError(f"gemm_skinny_gelu_row: bfloat16 x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
+    if x.stride(1) != 1 or w.stride(1) != 1 or out.stride(1) != 1:
+        raise KernelError("gemm_skinny_gelu_row: innermost dimension must be contiguous")
+    f = _fn("gemm_skinny", "il_gemm_skinny_gelu_row", [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p,
+                                                       _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p])
+    _check(f(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(out), out.stride(0), M, N, K, _ptr(ids), _ptr(table), table.stride(0), off, dim,
+             table.shape[0], _stream()), "gemm_skinny_gelu_row")
 
 
 def add_bias(y: torch.Tensor, bias: torch.Tensor) -> None:
@@ -217,15 +265,17 @@ def rope_store(qkv: torch.Tensor, tok_pos: torch.Tensor, tok_entry: torch.Tensor
 def attention_plain(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                     tok_pos: torch.Tensor, tok_entry: torch.Tensor, page_size: int, n_heads: int,
                     n_kv_heads: int, head_dim: int, scale: float, window: Optional[int] = None,
-                    sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None, sigmoid: bool = False) -> None:
+                    sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None, sigmoid: bool = False,
+                    cap: Optional[float] = None) -> None:
     """Causal attention of every token of `qkv` over its request's cache pages (plain kernel). `qkv` needs the query
     heads only (keys and values are read from the cache). `sink`: float32 [heads], a score per head that joins the
     softmax's denominator without a value. `dist_bias`: float32 [far + 1, heads], added to the scaled score of a key n
     positions back as dist_bias[min(n, far), head]. `sigmoid`: a key's weight is the sigmoid of its score, not normalised over
-    the keys (no softmax, so no sink)."""
+    the keys (no softmax, so no sink). `cap`: the scaled score s becomes cap * tanh(s / cap) before the softmax (not the sink)."""
     _need_cuda(qkv, out, cache, block_table, tok_pos, tok_entry, sink, dist_bias)
     _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)
+    cap = _cap_arg(cap, dist_bias, sigmoid)
     T = qkv.shape[0]
     if out.shape != (T, n_heads * head_dim) or out.dtype != qkv.dtype or cache.dtype != qkv.dtype:
         raise KernelError("attention_plain: out [T, heads*head_dim], same dtype as qkv and cache")
@@ -234,11 +284,20 @@ def attention_plain(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, b
     _contig("qkv", qkv), _contig("out", out), _contig("cache", cache), _contig("block_table", block_table)
     f = _fn("attn_plain", "il_attn_plain", [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
                                             _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
-                                            _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p])
+                                            _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_float, _c_void_p])
     _check(f(_ptr(qkv), kind_of(qkv.dtype), qkv.shape[1], _ptr(out), _ptr(cache), _ptr(block_table),
              block_table.shape[1], _ptr(tok_pos), _ptr(tok_entry), page_size, T, n_heads, n_kv_heads, head_dim,
-             scale, int(window or 0), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), _stream()),
+             scale, int(window or 0), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), cap, _stream()),
            "attention_plain")
+
+
+def _cap_arg(cap: Optional[float], dist_bias: Optional[torch.Tensor], sigmoid: bool) -> float:
+    """The kernels' soft-cap argument: 0 for none."""
+    if cap is None:
+        return 0.0
+    if not float(cap) > 0.0 or dist_bias is not None or sigmoid:
+        raise KernelError("attention: a soft cap is positive and goes with softmax weights and no bias by distance")
+    return float(cap)
 
 
 def _check_sink(sink: Optional[torch.Tensor], n_heads: int, sigmoid: bool = False) -> None:
@@ -310,6 +369,56 @@ def norm_add_norm(resid: torch.Tensor, branch, branch_weight: torch.Tensor, bran
              kind_of(y.dtype), T, H, _stream()), "norm_add_norm")
 
 
+class BranchTerm:
+    """One branch of a sum: scale * col_scale * y, or, with `norm_weight`, scale * col_scale * y / rms(y) * norm_weight
+    (rms with `eps` inside its root). `norm_weight` and `col_scale` are [H] vectors, float32 or bfloat16."""
+    __slots__ = ("y", "scale", "norm_weight", "eps", "col_scale")
+
+    def __init__(self, y: torch.Tensor, scale: float = 1.0, norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                 col_scale: Optional[torch.Tensor] = None):
+        self.y, self.scale, self.norm_weight, self.eps, self.col_scale = y, float(scale), norm_weight, float(eps), col_scale
+
+
+BRANCH_MAX_TERMS = 4
+
+
+def branch_sum(terms, resid: Optional[torch.Tensor] = None, copy: Optional[torch.Tensor] = None, next_weight: Optional[torch.Tensor] = None,
+               next_eps: float = 0.0, out: Optional[torch.Tensor] = None) -> None:
+    """The sum of up to four `BranchTerm`s, made in float32: added into `resid` (float32 [T,H], in place); `copy` receives the new
+    rows of resid - the sum itself where there is no resid - and `out` = RMSNorm(resid) * next_weight, both in the branches' dtype."""
+    n = len(terms)
+    if not 0 < n <= BRANCH_MAX_TERMS or (resid is None and copy is None) or (out is not None and (next_weight is None or resid is None)):
+        raise KernelError(f"branch_sum: 1 to {BRANCH_MAX_TERMS} branches, and a resid or a copy; out comes with resid and next_weight")
+    T, H = terms[0].y.shape
+    dt = terms[0].y.dtype
+    _need_cuda(resid, copy, next_weight, out)
+    if len({t.y.data_ptr() for t in terms}) != n:
+        raise KernelError("branch_sum: two branches in one buffer")
+    for t in terms:
+        _need_cuda(t.y, t.norm_weight, t.col_scale)
+        if tuple(t.y.shape) != (T, H) or t.y.dtype != dt or not t.y.is_contiguous():
+            raise KernelError("branch_sum: branches [T,H] of one dtype, contiguous")
+        for v in (t.norm_weight, t.col_scale):
+            if v is not None and (v.numel() != H or not v.is_contiguous()):
+                raise KernelError("branch_sum: norm weights and column factors [H]")
+    if resid is not None and (resid.dtype != torch.float32 or tuple(resid.shape) != (T, H) or not resid.is_contiguous()):
+        raise KernelError("branch_sum: resid float32 [T,H]")
+    for v in (copy, out):
+        if v is not None and (v.dtype != dt or tuple(v.shape) != (T, H) or not v.is_contiguous()):
+            raise KernelError("branch_sum: copy and out [T,H] of the branches' dtype")
+    if next_weight is not None and (next_weight.numel() != H or not next_weight.is_contiguous()):
+        raise KernelError("branch_sum: next_weight [H]")
+    vp, ci, cf = _c_void_p * n, _c_int * n, _c_float * n
+
+    def kinds(name):
+        return ci(*[0 if getattr(t, name) is None else kind_of(getattr(t, name).dtype) for t in terms])
+    f = _fn("rmsnorm", "il_branch_sum", [_c_void_p] * 8 + [_c_int, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_void_p])
+    _check(f(_ptr(resid), vp(*[t.y.data_ptr() for t in terms]), vp(*[_ptr(t.norm_weight) for t in terms]), kinds("norm_weight"),
+             vp(*[_ptr(t.col_scale) for t in terms]), kinds("col_scale"), cf(*[t.scale for t in terms]), cf(*[t.eps for t in terms]), n,
+             _ptr(copy), _ptr(next_weight if out is not None else None), kind_of(next_weight.dtype) if out is not None else 0, next_eps, _ptr(out),
+             kind_of(dt), T, H, _stream()), "branch_sum")
+
+
 HYPER_MAX_STREAMS = 16
 
 
@@ -361,17 +470,23 @@ def cast_rows(x: torch.Tensor, out: torch.Tensor) -> None:
 def qk_norm_store(proj: torch.Tensor, q_off: int, k_off: Optional[int], v_off: int, n_heads: int, n_kv_heads: int, qk_dim: int, v_dim: int,
                   head_dim: int, w_q: torch.Tensor, w_k: Optional[torch.Tensor], eps: float, temp_coef: float, temp_every: int,
                   q_out: torch.Tensor, tok_pos: torch.Tensor, tok_entry: torch.Tensor, block_table: torch.Tensor,
-                  cache: Optional[torch.Tensor], page_size: int, bias: Optional[torch.Tensor] = None) -> None:
+                  cache: Optional[torch.Tensor], page_size: int, bias: Optional[torch.Tensor] = None,
+                  first: Optional[torch.Tensor] = None, mix: float = 0.0) -> None:
     """Per token and head: q / rms(q) * w_q (times 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1) if temp_every > 0)
     to `q_out` [T, heads * head_dim]; k / rms(k) * w_k to the K plane of the token's cache slot and the value columns (at
     `v_off`; the key columns themselves where the values are the keys as projected) to the V plane. Heads are laid out at
     head_dim >= qk_dim, v_dim, the surplus zero. `k_off` None: the mixer has no keys of its own, only queries are normed.
-    `bias`: float32, one number per column of `proj`, added to q, k and v before anything else."""
+    `bias`: float32, one number per column of `proj`, added to q, k and v before anything else.
+    `first` [T, kv_heads * v_dim] (a view with a row stride): the values stored are (1 - mix) v + mix first, in float32 up to the store."""
     _need_cuda(proj, w_q, w_k, q_out, tok_pos, tok_entry, block_table, cache, bias)
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != proj.shape[1] or not bias.is_contiguous()):
         raise KernelError("qk_norm_store: bias float32, one per column of proj")
     T = proj.shape[0]
     has_k = k_off is not None
+    if first is not None:
+        _need_cuda(first)
+        if not has_k or first.dtype != proj.dtype or tuple(first.shape) != (T, n_kv_heads * v_dim) or first.stride(1) != 1:
+            raise KernelError("qk_norm_store: first [T, kv_heads * v_dim] of proj's dtype, for a mixer with values of its own")
     if proj.stride(1) != 1 or q_off + n_heads * qk_dim > proj.shape[1] or (has_k and (k_off + n_kv_heads * qk_dim > proj.shape[1]
                                                                                     or v_off + n_kv_heads * v_dim > proj.shape[1])):
         raise KernelError("qk_norm_store: segments lie outside the rows")
@@ -387,20 +502,26 @@ def qk_norm_store(proj: torch.Tensor, q_off: int, k_off: Optional[int], v_off: i
             raise KernelError("qk_norm_store: cache [pages,2,kv_heads,page,head_dim] of proj's dtype")
     f = _fn("qk_norm", "il_qk_norm_store", [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                             _c_void_p, _c_void_p, _c_int, _c_float, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p,
-                                            _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p])
+                                            _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p])
     _check(f(_ptr(proj), kind_of(proj.dtype), proj.stride(0), q_off, k_off if has_k else -1, v_off, n_heads, n_kv_heads, qk_dim, v_dim,
              head_dim, _ptr(w_q), _ptr(w_k), kind_of(w_q.dtype), eps, temp_coef, temp_every, _ptr(q_out), _ptr(tok_pos), _ptr(tok_entry),
-             _ptr(block_table), block_table.shape[1], _ptr(cache if has_k else None), page_size, T, _ptr(bias), _stream()), "qk_norm_store")
+             _ptr(block_table), block_table.shape[1], _ptr(cache if has_k else None), page_size, T, _ptr(bias),
+             _ptr(first), 0 if first is None else first.stride(0), mix, _stream()), "qk_norm_store")
 
 
 def qk_rows_norm_rope_store(proj: torch.Tensor, q_off: int, k_off: Optional[int], v_off: int, n_heads: int, n_kv_heads: int, qk_dim: int,
                             v_dim: int, head_dim: int, w_q: torch.Tensor, w_k: Optional[torch.Tensor], eps: float, rot_dim: int,
                             inv_freq: Optional[torch.Tensor], q_out: torch.Tensor, tok_pos: torch.Tensor, tok_entry: torch.Tensor,
-                            block_table: torch.Tensor, cache: Optional[torch.Tensor], page_size: int) -> None:
+                            block_table: torch.Tensor, cache: Optional[torch.Tensor], page_size: int,
+                            pair_freq: Optional[torch.Tensor] = None) -> None:
     """Per token: all query columns are divided by their common root mean square and multiplied by `w_q` [heads * qk_dim], all
     key columns likewise with `w_k` [kv_heads * qk_dim]; then the first `rot_dim` dimensions of every head turn by
     pos * inv_freq[i] (dimension i paired with i + rot_dim / 2). Queries to `q_out` [T, heads * head_dim], keys and values to
-    the K and V plane of the token's cache slot; heads laid out at head_dim, the surplus zero. `k_off` None: queries only."""
+    the K and V plane of the token's cache slot; heads laid out at head_dim, the surplus zero. `k_off` None: queries only.
+    `pair_freq` (float64 [rot_dim / 2], instead of inv_freq): dimension 2i turns with 2i + 1, its angle made in double precision."""
+    _need_cuda(pair_freq)
+    if pair_freq is not None and (pair_freq.dtype != torch.float64 or pair_freq.numel() != rot_dim // 2 or not pair_freq.is_contiguous() or rot_dim == 0):
+        raise KernelError("qk_rows_norm_rope_store: pair_freq float64 [rot_dim / 2]")
     _need_cuda(proj, w_q, w_k, inv_freq, q_out, tok_pos, tok_entry, block_table, cache)
     T = proj.shape[0]
     has_k = k_off is not None
@@ -409,7 +530,9 @@ def qk_rows_norm_rope_store(proj: torch.Tensor, q_off: int, k_off: Optional[int]
         raise KernelError("qk_rows_norm_rope_store: segments lie outside the rows")
     if w_q.numel() != n_heads * qk_dim or (has_k and (w_k is None or w_k.numel() != n_kv_heads * qk_dim or w_k.dtype != w_q.dtype)):
         raise KernelError("qk_rows_norm_rope_store: norm weights of heads * qk_dim (queries) and kv_heads * qk_dim (keys) entries, one dtype")
-    if rot_dim and (inv_freq is None or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dim // 2 or rot_dim % 2 or rot_dim > qk_dim):
+    if rot_dim and (rot_dim % 2 or rot_dim > qk_dim):
+        raise KernelError("qk_rows_norm_rope_store: rot_dim even and at most qk_dim")
+    if rot_dim and pair_freq is None and (inv_freq is None or inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dim // 2 or rot_dim % 2 or rot_dim > qk_dim):
         raise KernelError("qk_rows_norm_rope_store: inv_freq float32 [rot_dim / 2], rot_dim even and at most qk_dim")
     if tuple(q_out.shape) != (T, n_heads * head_dim) or q_out.dtype != proj.dtype or not q_out.is_contiguous():
         raise KernelError("qk_rows_norm_rope_store: q_out [T, heads * head_dim] of proj's dtype")
@@ -420,11 +543,11 @@ def qk_rows_norm_rope_store(proj: torch.Tensor, q_off: int, k_off: Optional[int]
             raise KernelError("qk_rows_norm_rope_store: cache [pages,2,kv_heads,page,head_dim] of proj's dtype")
     f = _fn("qk_norm", "il_qk_rows_norm_rope_store", [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                                       _c_void_p, _c_void_p, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
-                                                      _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p])
+                                                      _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p])
     _check(f(_ptr(proj), kind_of(proj.dtype), proj.stride(0), q_off, k_off if has_k else -1, v_off, n_heads, n_kv_heads, qk_dim, v_dim,
-             head_dim, _ptr(w_q), _ptr(w_k), kind_of(w_q.dtype), eps, rot_dim, _ptr(inv_freq if rot_dim else None), _ptr(q_out),
+             head_dim, _ptr(w_q), _ptr(w_k), kind_of(w_q.dtype), eps, rot_dim, _ptr(inv_freq if rot_dim and pair_freq is None else None), _ptr(q_out),
              _ptr(tok_pos), _ptr(tok_entry), _ptr(block_table), block_table.shape[1], _ptr(cache if has_k else None), page_size, T,
-             _stream()), "qk_rows_norm_rope_store")
+             _ptr(pair_freq), _stream()), "qk_rows_norm_rope_store")
 
 
 def gate_pack(y: torch.Tensor, head_dim: int, gate: Optional[torch.Tensor], g_off: int, out: torch.Tensor, n_heads: int, v_dim: int) -> None:
@@ -495,7 +618,7 @@ def attention_decode(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
                      head_dim: int, scale: float, window: Optional[int], pages_per_split: int, n_splits: int,
                      o_part: torch.Tensor, ml_part: torch.Tensor, kv_map: Optional[torch.Tensor] = None,
                      sink: Optional[torch.Tensor] = None, v_is_k: bool = False, dist_bias: Optional[torch.Tensor] = None,
-                     sigmoid: bool = False) -> None:
+                     sigmoid: bool = False, cap: Optional[float] = None) -> None:
     """bfloat16 split-KV attention of token rows [0, n_decode) (entry i = row i, one token each), then the merge of
     the splits (a second launch; with n_splits = 1 there is none and the attention kernel writes `out` itself). A row whose length is 0 gets zeros; a block-table entry below 0 is never followed.
     pages_per_split 0: each request's pages are divided evenly over the n_splits splits.
@@ -503,10 +626,12 @@ def attention_decode(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
     v_is_k: the caller vouches that the V plane of every page repeats its K plane (a latent that is key and value at once);
     with a tensor map only the K plane is then read, half the bytes.
     sigmoid: a key's weight is the sigmoid of its score, not normalised over the keys.
+    cap: the scaled score s becomes cap * tanh(s / cap) before the softmax.
     Scratch: o_part float32 [n_decode*heads*n_splits*head_dim], ml_part float32 [n_decode*heads*n_splits*2]."""
     _need_cuda(qkv, out, cache, block_table, entry_kvlen, o_part, ml_part, sink, dist_bias)
     _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)      # float32 [far + 1, heads]: added to the scaled score of a key n positions back
+    cap = _cap_arg(cap, dist_bias, sigmoid)
     if qkv.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16:
         raise KernelError("attention_decode: bfloat16 tensors")
     if o_part is None or ml_part is None or o_part.dtype != torch.float32 or ml_part.dtype != torch.float32:
@@ -521,14 +646,14 @@ def attention_decode(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, 
     _contig("qkv", qkv), _contig("out", out), _contig("cache", cache), _contig("block_table", block_table)
     f = _fn("attn_decode", "il_attn_decode", [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int,
                                               _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_void_p,
-                                              _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p],
+                                              _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_float, _c_void_p],
             defines={"HEAD_DIM": head_dim})
     if kv_map is not None and (kv_map.is_cuda or kv_map.dtype != torch.uint8 or kv_map.numel() != KV_MAP_BYTES):
         raise KernelError("attention_decode: kv_map must be the host tensor kv_tensor_map returned")
     _check(f(_ptr(qkv), qkv.shape[1], _ptr(out), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(entry_kvlen),
              page_size, n_decode, n_heads, n_kv_heads, head_dim, scale, int(window or 0), pages_per_split, n_splits,
              _ptr(o_part), _ptr(ml_part), _ptr(kv_map), _ptr(stream_status(qkv.device)) if kv_map is not None else _c_void_p(0),
-             _ptr(sink), 1 if v_is_k else 0, _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), _stream()), "attention_decode")
+             _ptr(sink), 1 if v_is_k else 0, _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), cap, _stream()), "attention_decode")
     if n_splits > 1:
         count_launches(1)                         # the merge kernel (a single split needs none: the attention kernel finishes the rows)
 
@@ -575,12 +700,13 @@ def attention_prefill(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor,
                       entry_qstart: torch.Tensor, entry_kvlen: torch.Tensor, first_entry: int, n_entries: int,
                       n_tiles_total: int, page_size: int, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                       window: Optional[int], sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
-                      sigmoid: bool = False) -> None:
+                      sigmoid: bool = False, cap: Optional[float] = None) -> None:
     """bfloat16 causal attention of the tokens of entries [first_entry, n_entries) over their cache pages.
     n_tiles_total = sum over those entries of ceil(q_len / (64 // (heads/kv_heads)))."""
     _need_cuda(qkv, out, cache, block_table, entry_qstart, entry_kvlen, sink, dist_bias)
     _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)
+    cap = _cap_arg(cap, dist_bias, sigmoid)
     if qkv.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16:
         raise KernelError("attention_prefill: bfloat16 tensors")
     if out.shape != (qkv.shape[0], n_heads * head_dim):
@@ -588,10 +714,10 @@ def attention_prefill(qkv: torch.Tensor, out: torch.Tensor, cache: torch.Tensor,
     _contig("qkv", qkv), _contig("out", out), _contig("cache", cache), _contig("block_table", block_table)
     f = _fn("attn_prefill", "il_attn_prefill", [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p,
                                                 _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
-                                                _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p], defines={"HEAD_DIM": head_dim})
+                                                _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_float, _c_void_p], defines={"HEAD_DIM": head_dim})
     _check(f(_ptr(qkv), qkv.shape[1], _ptr(out), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(entry_qstart),
              _ptr(entry_kvlen), page_size, first_entry, n_entries, n_tiles_total, n_heads, n_kv_heads, head_dim, scale,
-             int(window or 0), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), _stream()), "attention_prefill")
+             int(window or 0), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1, int(sigmoid), cap, _stream()), "attention_prefill")
 
 
 _tc5_prefill_rows = {}
@@ -630,7 +756,7 @@ def attention_prefill_tc5(qkv: torch.Tensor, out: torch.Tensor, kv_map: torch.Te
                           entry_qstart: torch.Tensor, entry_kvlen: torch.Tensor, first_entry: int, n_entries: int,
                           n_tiles_total: int, page_size: int, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                           window: Optional[int], sink: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
-                          sigmoid: bool = False, log_bias: Optional[torch.Tensor] = None) -> None:
+                          sigmoid: bool = False, log_bias: Optional[torch.Tensor] = None, cap: Optional[float] = None) -> None:
     """The same attention as `attention_prefill`, on tcgen05 tensor cores with tensor memory; `kv_map` is the cache's
     tensor map (`kv_tensor_map`). `log_bias` (with `sigmoid`, instead of dist_bias): float32 [3, heads] - r1, r2 and an offset pb:
     the scaled score of a key n positions back gets pb - r1 ln(1 + r2 n), computed as it is needed. n_tiles_total = sum over the entries of ceil(q_len / (prefill_tc5_rows(head_dim) // (heads/kv_heads)))."""
@@ -640,6 +766,7 @@ def attention_prefill_tc5(qkv: torch.Tensor, out: torch.Tensor, kv_map: torch.Te
         raise KernelError("attention_prefill_tc5: log_bias float32 [3, heads], with sigmoid weights and without dist_bias")
     _check_sink(sink, n_heads, sigmoid)
     _check_dist_bias(dist_bias, n_heads)
+    cap = _cap_arg(cap, dist_bias, sigmoid)
     if qkv.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise KernelError("attention_prefill_tc5: bfloat16 tensors")
     if not _has_third_map(kv_map):
@@ -649,11 +776,11 @@ def attention_prefill_tc5(qkv: torch.Tensor, out: torch.Tensor, kv_map: torch.Te
     _contig("qkv", qkv), _contig("out", out), _contig("block_table", block_table)
     f = _fn("attn_prefill_tc5", "il_attn_prefill_tc5",
             [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p], defines={"HEAD_DIM": head_dim})
+             _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_float, _c_void_p], defines={"HEAD_DIM": head_dim})
     _check(f(_ptr(qkv), qkv.shape[1], _ptr(out), _c_void_p(kv_map.data_ptr() + 256), _ptr(block_table), block_table.shape[1],
              _ptr(entry_qstart), _ptr(entry_kvlen), page_size, first_entry, n_entries, n_tiles_total, n_heads, n_kv_heads,
              head_dim, scale, int(window or 0), _ptr(stream_status(qkv.device)), _ptr(sink), _ptr(dist_bias), 0 if dist_bias is None else dist_bias.shape[0] - 1,
-             int(sigmoid), _ptr(log_bias), _stream()), "attention_prefill_tc5")
+             int(sigmoid), _ptr(log_bias), cap, _stream()), "attention_prefill_tc5")
 
 
 SKINNY_MAX_ROWS = 16
@@ -718,11 +845,12 @@ def _norm_args(norm_in: Optional[NormedInput], M: int):
 def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, alpha: float = 1.0,
                 bias: Optional[torch.Tensor] = None, glu: int = 0, norm_in: Optional[NormedInput] = None, act_params=None) -> None:
     """out[M,N] = alpha * x[M,K] @ w[N,K]^T (+ bias) for M <= 16 bfloat16 rows; out bfloat16 or float32.
-    glu (True, or ACT_SILU / ACT_GELU_TANH / ACT_CLAMPED with act_params): w is [2N,K] (gate rows, then up rows) and out[M,N] = act(gate) * up.
+    glu (True, or ACT_SILU / ACT_GELU_TANH / ACT_CLAMPED with act_params): w is [2N,K] (gate rows, then up rows) and out[M,N] = act(gate) * up;
+    ACT_RELU2: w is [N,K] and out is relu(.)^2 of the product (bfloat16).
     norm_in: x is `norm_in.xw`, and the results are divided by the rms that its sums give."""
     _need_cuda(x, w, out, bias)
     M, K = x.shape
-    N = w.shape[0] // 2 if glu else w.shape[0]
+    N = w.shape[0] // 2 if glu and int(glu) != ACT_RELU2 else w.shape[0]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != K or out.shape != (M, N):
         raise KernelError(f"gemm_skinny: bfloat16 x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
     if x.stride(1) != 1 or w.stride(1) != 1 or out.stride(1) != 1:
@@ -888,10 +1016,11 @@ def gemm_mid(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, alpha: float =
              glu: int = 0, nb: int = 0, bm: int = 0, act_params=None) -> None:
     """out[M,N] = alpha * x[M,K] @ w[N,K]^T (+ bias) for 17..128 bfloat16 rows on the tcgen05 tensor cores: tiles of 64
     or 128 weight rows (`bm`; the A operand) by blocks of `nb` activation rows (0: chosen by the kernel) over all of K; out bfloat16
-    or float32. glu (True, or ACT_SILU / ACT_GELU_TANH / ACT_CLAMPED with act_params): w is [2N,K] (gate rows, then up rows) and out[M,N] = act(gate) * up (bfloat16)."""
+    or float32. glu (True, or ACT_SILU / ACT_GELU_TANH / ACT_CLAMPED with act_params): w is [2N,K] (gate rows, then up rows) and out[M,N] = act(gate) * up (bfloat16);
+    ACT_RELU2: w is [N,K], out relu(.)^2 of the product (bfloat16)."""
     _need_cuda(x, w, out, bias)
     M, K = x.shape
-    N = w.shape[0] // 2 if glu else w.shape[0]
+    N = w.shape[0] // 2 if glu and int(glu) != ACT_RELU2 else w.shape[0]
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != K or out.shape != (M, N):
         raise KernelError(f"gemm_mid: bfloat16 x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
     if x.stride(1) != 1 or w.stride(1) != 1 or out.stride(1) != 1:

@@ -32,6 +32,7 @@ class PagedAttend:
     `chunk`: instead of a sliding window, runs of `chunk` positions counted from position 0 of the sequence; a query sees the
     keys of its own run up to itself (the kernels take it as a negative window). The cache keeps every page: a window's
     pages are given back behind it, a chunked layer's are not (another layer may read them).
+    `cap`: the scaled score s becomes cap * tanh(s / cap) before the softmax (a sink is not capped).
     `sigmoid`: no softmax - a visible key's weight is the sigmoid of its score (scaled, biased), not normalised over the keys.
     `log_bias`: float32 [3, heads] on the device or None - the numbers r1, r2, pb whose pb - r1 ln(1 + r2 n) `dist_bias` holds by
     distance: a kernel that would rather compute than look up takes these (sigmoid weights on the tensor-memory prefill kernel)."""
@@ -46,7 +47,7 @@ class PagedAttend:
 
     def __init__(self, dtype, n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: Optional[int] = None,
                  force_plain: bool = False, prefill_kernel: str = "auto", shared_kv: bool = False, chunk: Optional[int] = None,
-                 sigmoid: bool = False):
+                 sigmoid: bool = False, cap: Optional[float] = None):
         if chunk is not None and (window is not None or int(chunk) < 1):
             raise ValueError("attention: a mask is a window or runs of a positive size, not both")
         self.dtype, self.nh, self.nkv, self.hd, self.scale, self.window = dtype, n_heads, n_kv_heads, head_dim, scale, window
@@ -54,7 +55,9 @@ class PagedAttend:
         self.span = self.chunk if self.chunk is not None else window          # the most keys a query sees (None: all)
         self.mask_arg = -self.chunk if self.chunk is not None else window     # what the kernels take
         self.force_plain, self.prefill_kernel, self.shared_kv = force_plain, prefill_kernel, shared_kv
-        self.sigmoid = bool(sigmoid)
+        self.sigmoid, self.cap = bool(sigmoid), None if cap is None else float(cap)
+        if self.cap is not None and not self.cap > 0.0:
+            raise ValueError("attention: a soft cap on the scores is positive")
         self.sink: Optional[torch.Tensor] = None
         self.dist_bias: Optional[torch.Tensor] = None
         self.log_bias: Optional[torch.Tensor] = None
@@ -80,7 +83,8 @@ class PagedAttend:
                               "head sizes in steps of 16 up to 256): the plain kernel runs, at a fraction of their speed",
                               RuntimeWarning, stacklevel=2)
             ops.attention_plain(qkv, out, cache.storage, cache.block_table, ctx.tok_pos, ctx.tok_entry,
-                                cache.page_size, self.nh, self.nkv, self.hd, self.scale, self.mask_arg, self.sink, self.dist_bias, self.sigmoid)
+                                cache.page_size, self.nh, self.nkv, self.hd, self.scale, self.mask_arg, self.sink, self.dist_bias, self.sigmoid,
+                                self.cap)
             return
         n_dec, E = ctx.n_decode, ctx.n_entries
         if n_dec > 0:
@@ -96,7 +100,7 @@ class PagedAttend:
                                  self.nh, self.nkv, self.hd, self.scale, self.mask_arg, 0, n_splits,
                                  ctx.ws.flat("attn_o_part", rows * self.hd, torch.float32),
                                  ctx.ws.flat("attn_ml_part", rows * 2, torch.float32), kv_map=cache.tma_map, sink=self.sink,
-                                 v_is_k=v_is_k, dist_bias=self.dist_bias, sigmoid=self.sigmoid)
+                                 v_is_k=v_is_k, dist_bias=self.dist_bias, sigmoid=self.sigmoid, cap=self.cap)
         if E > n_dec:
             # prompt portions: on tcgen05 with tensor memory where the head size has that kernel (64, 128, 256) and the cache
             # its tensor map; else the mma.sync kernel. The tile is 128 (64) rows = tokens x heads of a kv head.
@@ -108,11 +112,11 @@ class PagedAttend:
                 ops.attention_prefill_tc5(qkv, out, cache.tma_map, cache.block_table, ctx.entry_qstart, ctx.entry_kvlen,
                                           n_dec, E, n_tiles, cache.page_size, self.nh, self.nkv, self.hd, self.scale,
                                           self.mask_arg, sink=self.sink, dist_bias=self.dist_bias if self.log_bias is None else None,
-                                          sigmoid=self.sigmoid, log_bias=self.log_bias)
+                                          sigmoid=self.sigmoid, log_bias=self.log_bias, cap=self.cap)
             else:
                 ops.attention_prefill(qkv, out, cache.storage, cache.block_table, ctx.entry_qstart, ctx.entry_kvlen,
                                       n_dec, E, n_tiles, cache.page_size, self.nh, self.nkv, self.hd, self.scale,
-                                      self.mask_arg, sink=self.sink, dist_bias=self.dist_bias, sigmoid=self.sigmoid)
+                                      self.mask_arg, sink=self.sink, dist_bias=self.dist_bias, sigmoid=self.sigmoid, cap=self.cap)
 
 
 class Attention(Mixer):

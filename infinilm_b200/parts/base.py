@@ -102,6 +102,9 @@ class Mixer(Part):
     def fuses_tail(self, T: int) -> bool:
         return False
 
+    # True: `forward(..., terms=True)` returns a list of `ops.BranchTerm`s for a reader that sums the mixer's branches itself
+    gives_terms = False
+
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
         """x [T,H] in the compute dtype -> y [T,H]. `cache` is this run entry's view of the cache
         (`PagedKVView`, `StateView` or None); `cache.writable` is False when the entry reads
@@ -140,6 +143,10 @@ class Arrangement:
         block accepts a normed input; it may then return an `ops.NormedInput` for it. An arrangement with `takes_pre_add`
         has the argument `pre_add=None`: a float32 [H] vector to add to the residual stream before its first norm."""
         raise NotImplementedError
+
+    one_norm = False                             # True: both sublayers read one norm's output (the layer names no norm for the feed-forward)
+
+    takes_token_table = False                    # True: `set_token_table(part)` receives the model's table of per-layer token rows
 
     takes_pre_add = False                        # True: `run` has the `pre_add` argument
 
@@ -189,4 +196,4 @@ def _ensure_builtin() -> None:
     if not _builtin_done:
         _builtin_done = True
         from . import (attention, blocks, conv_attention, embedding, feed_forward, latent_attention, linear_recurrence, moe, normed_attention,  # noqa: F401
-                       norms, parallel, position)
+                       norms, parallel, position, token_input)

@@ -16,6 +16,7 @@ import torch
 from .. import ops
 from .base import Arrangement, Part, ResidualTail, build_part, register_part
 from .spec import WeightSpec
+from .token_input import TokenInput
 
 
 class PreNormResidual(Arrangement):
@@ -145,6 +146,96 @@ class SandwichResidual(Arrangement):
         return ops.StreamDone(None if nxt is None else normed)
 
 
+class BranchScales(Part):
+    """A factor per column on what a block's sublayers return, before it joins the stream: ls1 [hidden] on the mixer's result, ls2 on
+    the feed-forward's (which a layer without one need not have). params: hidden, sublayers."""
+    graph_safe = True
+
+    def __init__(self, params, prefix, dtype):
+        super().__init__(params, prefix, dtype)
+        self.hidden, self.n_sub = int(params["hidden"]), int(params["sublayers"])
+        self.w: List[torch.Tensor] = []
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [WeightSpec(f"ls{q}", (self.hidden,), "vector", ("ones_normal", 0.1), optional=q > self.n_sub) for q in (1, 2)]
+
+    def set_weights(self, t: Dict[str, torch.Tensor]) -> None:
+        self.w = [t[f"ls{q}"].contiguous() for q in range(1, self.n_sub + 1)]
+
+
+class ParallelResidual(Arrangement):
+    """h = norm(x); x <- x + (s1 * mixer(h) + s2 * ffn(h)): both sublayers read one norm's output and join the stream together, each
+    under an optional factor per column; then, optionally, the layer's own token input (`parts/token_input.py`).
+    params: scales (None, or the prefix of the layer's ls1 and ls2), token_input (None or a PartSpec's params and prefix).
+    One kernel adds all branches - a parallel mixer's come to it unsummed, with their norms - and leaves the stream's copy in the
+    compute dtype for the token input's gate; one more adds the token input's normed branch and makes the next block's norm.
+    Without a token input the first of the two makes the next norm."""
+
+    one_norm = True
+    takes_next_block = True
+    takes_token_table = True
+
+    def __init__(self, mixer_norm, mixer, ffn_norm, ffn, params):
+        super().__init__(mixer_norm, mixer, ffn_norm, ffn, params)
+        if not mixer_norm.fusable_rms:
+            raise ValueError("a block whose sublayers run side by side takes an RMS norm")
+        hidden, dt = mixer_norm.size, mixer_norm.dtype
+        self.scales = None
+        if params.get("scales") is not None:
+            self.scales = BranchScales({"hidden": hidden, "sublayers": 1 if ffn is None else 2}, str(params["scales"]), dt)
+        ti = params.get("token_input")
+        self.token_input = None if ti is None else TokenInput(ti.params, ti.prefix, dt)
+        self.table = None
+
+    def set_token_table(self, table) -> None:
+        ti = self.token_input
+        if ti is not None and (table is None or ti.offset + ti.dim > table.width):
+            raise ValueError("a layer with a token input needs a token table with columns for it")
+        self.table = table
+
+    def parts(self):
+        return super().parts() + [p for p in (self.scales, self.token_input) if p is not None]
+
+    def run(self, resid, pending, ctx, cache, next_block=None):
+        T, H = resid.shape
+        if isinstance(pending, ops.NormedInput):
+            raise ValueError("a block whose sublayers run side by side cannot take a half-done norm")
+        normed = ctx.ws.rows("normed", T, H, ctx.dtype)
+        if isinstance(pending, ops.StreamDone) and pending.normed is not None:
+            normed = pending.normed
+        else:
+            branch, bscale = pending if isinstance(pending, tuple) else (None, 1.0)
+            self.mixer_norm.add_norm(resid, branch, bscale, normed)
+        if self.mixer.gives_terms:
+            terms = self.mixer.forward(normed, ctx, cache, terms=True)
+        else:
+            terms = [ops.BranchTerm(self.mixer.forward(normed, ctx, cache))]
+        ls = self.scales.w if self.scales is not None else (None, None)
+        for t in terms:
+            t.col_scale = ls[0]
+        if self.ffn is not None:
+            terms.append(ops.BranchTerm(self.ffn.forward(normed, ctx), col_scale=ls[1]))
+        nxt = next_block if isinstance(next_block, ParallelResidual) else None
+        while len(terms) > ops.BRANCH_MAX_TERMS:  # (more branches than one launch takes)
+            ops.branch_sum(terms[:ops.BRANCH_MAX_TERMS], resid)
+            terms = terms[ops.BRANCH_MAX_TERMS:]
+        if self.token_input is None:
+            if nxt is None:
+                ops.branch_sum(terms, resid)
+            else:
+                ops.branch_sum(terms, resid, next_weight=nxt.mixer_norm.weight, next_eps=nxt.mixer_norm.eps, out=normed)
+        else:
+            copy = None if ctx.dtype == torch.float32 else ctx.ws.rows("stream_copy", T, H, ctx.dtype)
+            ops.branch_sum(terms, resid, copy=copy)
+            ti = self.token_input
+            y = ti.branch(resid if copy is None else copy, self.table.table, ctx)
+            if nxt is None:
+                ops.norm_add_norm(resid, y, ti.norm_w, ti.eps)
+            else:
+                ops.norm_add_norm(resid, y, ti.norm_w, ti.eps, nxt.mixer_norm.weight, nxt.mixer_norm.eps, normed)
+        return ops.StreamDone(None if nxt is None else normed)
+
+
 class StreamWeights(Part):
     """The numbers by which a block with several copies of the residual stream reads and writes them, per sublayer q (1: the
     mixer, 2: the feed-forward): hc<q>.in [S] (the sublayer's input is sum_s in[s] x_s), hc<q>.mix [S, S] (from, to) and
@@ -233,3 +324,4 @@ register_part("arrangement", "prenorm_residual", PreNormResidual)
 register_part("arrangement", "hyper_connections", HyperConnections)
 register_part("arrangement", "branch_norm_residual", BranchNormResidual)
 register_part("arrangement", "sandwich_residual", SandwichResidual)
+register_part("arrangement", "parallel_residual", ParallelResidual)

@@ -143,6 +143,24 @@ class RowTable(Part):
         return self._rows[i]
 
 
+class TokenTable(Part):
+    """A table with a row of `width` numbers per token, of which every layer takes its own columns (`parts/token_input.py`).
+    params: vocab, width, name. Held in the compute dtype."""
+    graph_safe = True
+
+    def __init__(self, params, prefix, dtype):
+        super().__init__(params, prefix, dtype)
+        self.vocab, self.width, self.name = int(params["vocab"]), int(params["width"]), str(params.get("name", "weight"))
+        self.table: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [WeightSpec(self.name, (self.vocab, self.width), init=("normal", 1.0))]
+
+    def set_weights(self, t: Dict[str, torch.Tensor]) -> None:
+        self.table = t[self.name].to(self.dtype).contiguous()
+
+
+register_part("embedding", "token_table", TokenTable)
 register_part("embedding", "token_embedding", TokenEmbedding)
 register_part("embedding", "pair_position_embedding", PairPositionEmbedding)
 register_part("embedding", "row_table", RowTable)

@@ -1,4 +1,4 @@
-"""Dense gated feed-forward: down(act(gate(x)) * up(x)), act SiLU (SwiGLU) or the tanh form of GELU; or, "clamped", with
+"""Dense feed-forwards. Without a gate: down(relu(up(x))^2). Gated: down(act(gate(x)) * up(x)), act SiLU (SwiGLU) or the tanh form of GELU; or, "clamped", with
 g = min(gate(x), limit) and u = up(x) kept within -limit .. limit: down(g sigmoid(alpha g) (u + 1)).
 
 Parity with InfiniLM: `csrc/layers/mlp/mlp.cpp:7-38` (gate and up as one product, `swiglu(up, gate)`,
@@ -76,17 +76,61 @@ class SwiGLU(FeedForward):
                                              tail.norm.weight, tail.norm.eps,
                                              ctx.ws.rows("xw_ffn", T, self.hidden, self.dtype),
                                              ctx.ws.rows("sumsq_ffn", T, (self.hidden + 15) // 16, torch.float32))
-            return self.down(act, ctx.ws.rows("branch", T, self.hidden, self.dtype))
+            return self.down(act, ctx.ws.rows("ffn_branch", T, self.hidden, self.dtype))
         act = ctx.ws.rows("ffn_act", T, self.inter, self.dtype)
         if self.dtype == torch.bfloat16 and ops.mid_ok(T, self.hidden):
             # 17..128 rows: gate and up on the tcgen05 tensor cores as two accumulators in the same lanes, SiLU(gate)*up in
             # the epilogue (measured against the library product followed by the SwiGLU kernel at 8B sizes: 44.6 against
             # 48.4 us at 32 rows, 47.6 against 49.9 at 64, 52.5 against 57.6 at 128)
             ops.gemm_mid(x, self.gate_up.weight, act, 1.0, self.gate_up.bias, glu=self.act, act_params=self.act_params)
-            return self.down(act, ctx.ws.rows("branch", T, self.hidden, self.dtype))
+            return self.down(act, ctx.ws.rows("ffn_branch", T, self.hidden, self.dtype))
         gu = self.gate_up(x, ctx.ws.rows("gate_up", T, 2 * self.inter, self.dtype))
         ops.swiglu(gu, act, self.act, self.act_params)
-        return self.down(act, ctx.ws.rows("branch", T, self.hidden, self.dtype))
+        return self.down(act, ctx.ws.rows("ffn_branch", T, self.hidden, self.dtype))
+
+
+class SquaredReLU(FeedForward):
+    """down(relu(up(x))^2). params: hidden, intermediate, names (local tensor names of the two weights, default up_proj.weight /
+    down_proj.weight)."""
+    graph_safe = True
+
+    def __init__(self, params, prefix, dtype):
+        super().__init__(params, prefix, dtype)
+        self.hidden, self.inter = int(params["hidden"]), int(params["intermediate"])
+        names = params.get("names") or {}
+        self.n_up, self.n_down = str(names.get("up", "up_proj.weight")), str(names.get("down", "down_proj.weight"))
+        self.up, self.down = Linear(self.hidden, self.inter, dtype), Linear(self.inter, self.hidden, dtype)
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [WeightSpec(self.n_up, (self.inter, self.hidden)), WeightSpec(self.n_down, (self.hidden, self.inter))]
+
+    def set_weights(self, t: Dict[str, torch.Tensor]) -> None:
+        self.up.set(t[self.n_up])
+        self.down.set(t[self.n_down])
+
+    def accepts_normed(self, T):
+        return self.dtype == torch.bfloat16 and ops.skinny_ok(T, self.hidden)
+
+    def fuses_tail(self, T):
+        return self.dtype == torch.bfloat16 and ops.skinny_ok(T, self.hidden) and ops.skinny_resid_ok(T, self.inter, self.hidden)
+
+    def forward(self, x, ctx, tail=None):
+        T = x.shape[0]
+        act = ctx.ws.rows("ffn_act", T, self.inter, self.dtype)
+        if self.dtype == torch.bfloat16 and ops.skinny_ok(T, self.hidden):      # the activation in the product's epilogue
+            normed = isinstance(x, ops.NormedInput)
+            ops.gemm_skinny(x.xw if normed else x, self.up.weight, act, glu=ops.ACT_RELU2, norm_in=x if normed else None)
+        elif self.dtype == torch.bfloat16 and ops.mid_ok(T, self.hidden):
+            ops.gemm_mid(x, self.up.weight, act, glu=ops.ACT_RELU2)
+        else:
+            self.up(x, act)
+            ops.relu2(act, act)
+        if tail is not None:                      # down adds into the residual and prepares the next norm itself
+            return ops.gemm_skinny_resid(act, self.down.weight, self.down.alpha, self.down.bias, tail.resid, tail.scale,
+                                         tail.norm.weight, tail.norm.eps, ctx.ws.rows("xw_ffn", T, self.hidden, self.dtype),
+                                         ctx.ws.rows("sumsq_ffn", T, (self.hidden + 15) // 16, torch.float32))
+        return self.down(act, ctx.ws.rows("ffn_branch", T, self.hidden, self.dtype))
 
 
 register_part("feed_forward", "swiglu", SwiGLU)
+register_part("feed_forward", "squared_relu", SquaredReLU)

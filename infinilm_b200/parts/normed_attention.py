@@ -14,6 +14,12 @@ Another way to weigh the keys (`weights` "sigmoid"): no softmax, o_h = sum over 
 pb one number per head (tensor `pb`). Another bias by distance (`distance_log`): the score loses r1_h ln(1 + r2_h (i - j))
 (tensors `r1`, `r2` [heads]); over a window it is unrolled at load into the same table by distance, pb joining it.
 
+The softmax's denominator may hold a learned number per head (`sink` "learned", tensor `sink` [heads]: exp(sink), neither scaled nor
+capped); scores may be soft-capped (`score_cap`); the gate may be one number per head (`gate_per` "head"); rotary pairs may be
+neighbours (an `interleaved` encoding, with the norm over the projection). Values may be blended with those an earlier layer
+projected for the same token (`value_mix`): v <- (1 - vmix) v + vmix v_first (tensor `vmix`, one number); the blend is what the
+cache holds.
+
 Options: the values may be the keys as projected, before their norm (no v tensor); a mixer may read the keys and values that
 another run-order entry cached (no k, v tensors, no cache of its own); key size and value size may differ - heads are laid
 out at hd = max of the two rounded up to 16, the surplus columns zero, as `conv_attention` does.
@@ -61,7 +67,10 @@ class QKNormAttention(Mixer):
     position (PartSpec of a rotary encoding, with norm_over "projection"), chunk (runs of that many positions, counted from the
     sequence's start; a query sees its own run) or window (a sliding window; its pages are given back behind it);
     bias_in_norm (the projection's biases are added, in float32, by the kernel that norms; with a norm per head),
-    weights ("softmax", the default, or "sigmoid"), distance_log (with a window, instead of distance_bias)."""
+    weights ("softmax", the default, or "sigmoid"), distance_log (with a window, instead of distance_bias);
+    sink (None or "learned"), score_cap (None or c: score <- c tanh(score / c)), gate_per ("column", the default, or "head"),
+    value_mix (None or {"role": "first" or "later", "key": name}, with a norm per head: the first leaves its projected values in
+    the step's `shared` under that name, the later ones blend them in; every one of them has a tensor `vmix`)."""
     graph_safe = True
     MAX_DISTANCES = 1 << 20                       # rows of an unrolled table by distance
 
@@ -90,12 +99,19 @@ class QKNormAttention(Mixer):
         if qt and self.t_every < 1:
             raise ValueError("attention: the query temperature's step must be at least 1")
         self.sink_zero = bool(p.get("sink_zero", False))
+        sink = p.get("sink")
+        if sink not in (None, "learned") or (sink and self.sink_zero):
+            raise ValueError("attention: sink is None or 'learned', and one kind of sink is enough")
+        self.sink_learned = sink == "learned"
+        self.cap = None if p.get("score_cap") is None else float(p["score_cap"])
         kind = str(p.get("weights", "softmax"))
         if kind not in ("softmax", "sigmoid"):
             raise ValueError("attention: weights is 'softmax' or 'sigmoid'")
         self.sigmoid, self.dist_log = kind == "sigmoid", bool(p.get("distance_log", False))
-        if self.sigmoid and self.sink_zero:
+        if self.sigmoid and (self.sink_zero or self.sink_learned):
             raise ValueError("attention: a sink belongs to a softmax")
+        if self.cap is not None and (self.sigmoid or self.dist_log or self.has_bias):
+            raise ValueError("attention: capped scores go with softmax weights and no bias by distance")
         if (self.sigmoid or self.dist_log) and (self.has_bias or p.get("window") is None):
             raise ValueError("attention: sigmoid weights and a logarithmic bias by distance go with a window and without a learned table")
         if (self.sigmoid or self.dist_log) and int(p["window"]) > self.MAX_DISTANCES:
@@ -104,11 +120,20 @@ class QKNormAttention(Mixer):
         if str(p.get("norm_over", "head")) not in ("head", "projection"):
             raise ValueError("attention: norm_over is 'head' or 'projection'")
         self.position = build_part("position", p.get("position") or PartSpec("none"), dtype)
-        if self.position.interleaved or self.position.has_transform or (self.position.rot_dim and not self.norm_rows) or self.position.rot_dim > self.dk:
+        if self.position.has_transform or self.position.mscale != 1.0 or (self.position.rot_dim and not self.norm_rows) or self.position.rot_dim > self.dk:
             raise ValueError("attention: a rotary table of at most qk_dim dimensions, with the norm over the projection")
         if self.norm_rows and (self.v_from_k or qt):
             raise ValueError("attention: the norm over the projection goes with values of their own and no query temperature")
         self.window, self.chunk = p.get("window"), p.get("chunk")
+        per = str(p.get("gate_per", "column"))
+        if per not in ("column", "head"):
+            raise ValueError("attention: gate_per is 'column' or 'head'")
+        self.n_gate = 0 if not self.gate else self.nh if per == "head" else self.nh * self.dv
+        self.head_gate = self.gate and per == "head"
+        vm = p.get("value_mix")
+        self.mix_role, self.mix_key = (str(vm["role"]), str(vm["key"])) if vm else (None, None)
+        if vm and (self.mix_role not in ("first", "later") or self.norm_rows or self.v_from_k or not self.own_kv or self.qkv_bias):
+            raise ValueError("attention: value_mix is 'first' or 'later', with a norm per head, values of their own and no biases")
         # the projection's columns: [q | k | v | g], k and v only with a cache of its own, v only if it is not k
         self.nq, self.nk, self.nvv = self.nh * self.dk, self.nkv * self.dk, self.nkv * self.dv
         self.q_off, off = 0, self.nq
@@ -120,16 +145,17 @@ class QKNormAttention(Mixer):
             else:
                 self.v_off, off = off, off + self.nvv
         self.g_off = off
-        self.n_proj = off + (self.nh * self.dv if self.gate else 0)
+        self.n_proj = off + self.n_gate
         self.n_proj_pad = (self.n_proj + 7) // 8 * 8
         self.proj = Linear(self.hidden, self.n_proj_pad, dtype)
         self.o_proj = Linear(self.nh * self.dv, self.hidden, dtype)
         self.core = PagedAttend(dtype, self.nh, self.nkv, self.hd, self.scale, self.window, bool(p.get("plain_kernel", False)),
-                                str(p.get("prefill_kernel", "auto")), chunk=self.chunk, sigmoid=self.sigmoid)
+                                str(p.get("prefill_kernel", "auto")), chunk=self.chunk, sigmoid=self.sigmoid, cap=self.cap)
         self.bias_in_norm = bool(p.get("bias_in_norm", False)) and self.qkv_bias
         if self.bias_in_norm and self.norm_rows:
             raise ValueError("attention: biases join in the norm's kernel where the norm is per head")
         self.w_q = self.w_k = self.bias = None
+        self.mix = 0.0
 
     def weight_specs(self) -> List[WeightSpec]:
         H = self.hidden
@@ -152,7 +178,11 @@ class QKNormAttention(Mixer):
         if self.sigmoid:
             specs.append(WeightSpec("pb", (self.nh,), "vector", ("normal", 1.0)))
         if self.gate:
-            specs.append(WeightSpec("g", (self.nh * self.dv, H)))
+            specs.append(WeightSpec("g", (self.n_gate, H)))
+        if self.sink_learned:
+            specs.append(WeightSpec("sink", (self.nh,), "vector", ("normal", 1.0)))
+        if self.mix_role:
+            specs.append(WeightSpec("vmix", (), "vector", ("normal", 0.5)))
         return specs
 
     def set_weights(self, t: Dict[str, torch.Tensor]) -> None:
@@ -188,6 +218,10 @@ class QKNormAttention(Mixer):
                 self.core.log_bias = torch.stack([t["r1"].float(), t["r2"].float(), t["pb"].float()]).contiguous()
         if self.sink_zero:
             self.core.sink = torch.zeros(self.nh, dtype=torch.float32, device=dev)
+        if self.sink_learned:
+            self.core.sink = t["sink"].to(torch.float32).contiguous()
+        if self.mix_role == "later":
+            self.mix = float(t["vmix"].float().item())
         self.position.to_device(dev)
 
     def cache_need(self) -> Optional[CacheNeed]:
@@ -198,21 +232,31 @@ class QKNormAttention(Mixer):
         T, hd = x.shape[0], self.hd
         if cache is None or (self.own_kv and not cache.writable) or (not self.own_kv and cache.writable):
             raise ValueError("attention: a mixer with keys of its own writes its cache; one without reads another entry's")
-        proj = self.proj(x, ctx.ws.rows("qna_proj", T, self.n_proj_pad, self.dtype))
+        # (the rows whose values later layers of the step read stay in a buffer of their own)
+        proj = self.proj(x, ctx.ws.rows(f"qna_proj_{self.mix_key}" if self.mix_role == "first" else "qna_proj", T, self.n_proj_pad, self.dtype))
+        first = None
+        if self.mix_role == "first":
+            ctx.shared[self.mix_key] = proj[:, self.v_off: self.v_off + self.nvv]
+        elif self.mix_role == "later":
+            first = ctx.shared[self.mix_key]
         q = ctx.ws.rows("qna_q", T, self.nh * hd, self.dtype)
         if self.norm_rows:
             ops.qk_rows_norm_rope_store(proj, self.q_off, self.k_off, self.v_off if self.own_kv else 0, self.nh, self.nkv, self.dk, self.dv, hd,
                                         self.w_q, self.w_k, self.eps, self.position.rot_dim, self.position.inv_freq, q, ctx.tok_pos,
-                                        ctx.tok_entry, cache.block_table, cache.storage if self.own_kv else None, cache.page_size)
+                                        ctx.tok_entry, cache.block_table, cache.storage if self.own_kv else None, cache.page_size,
+                                        pair_freq=self.position.freq64 if self.position.interleaved else None)
         else:
             ops.qk_norm_store(proj, self.q_off, self.k_off, self.v_off if self.own_kv else 0, self.nh, self.nkv, self.dk, self.dv, hd,
                               self.w_q, self.w_k, self.eps, self.t_coef, self.t_every, q, ctx.tok_pos, ctx.tok_entry, cache.block_table,
-                              cache.storage if self.own_kv else None, cache.page_size, bias=self.bias)
+                              cache.storage if self.own_kv else None, cache.page_size, bias=self.bias, first=first, mix=self.mix)
         att = ctx.ws.rows("qna_att", T, self.nh * hd, self.dtype)
         self.core.run(q, att, ctx, cache)
         if self.gate or hd != self.dv:
             gated = ctx.ws.rows("qna_gated", T, self.nh * self.dv, self.dtype)
-            ops.gate_pack(att, hd, proj if self.gate else None, self.g_off, gated, self.nh, self.dv)
+            if self.head_gate:
+                ops.head_gate(att, hd, proj, self.g_off, gated, self.nh, self.dv)
+            else:
+                ops.gate_pack(att, hd, proj if self.gate else None, self.g_off, gated, self.nh, self.dv)
             att = gated
         return self.o_proj(att, ctx.ws.rows("qna_branch", T, self.hidden, self.dtype))
 

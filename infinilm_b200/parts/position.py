@@ -1,4 +1,4 @@
-"""Rotary position encodings: plain RoPE, LongRoPE and YaRN, as frequency tables a mixer applies.
+"""Rotary position encodings: plain RoPE, LongRoPE, YaRN and Llama 3.1's scaling, as frequency tables a mixer applies.
 
 Parity with InfiniLM: `csrc/layers/rotary_embedding/rotary_embedding.cpp:50-113` (one rotary
 object from head_dim, rotary_dim, max positions, theta, scaling), `rope_scaling_creators.cpp:23-47`
@@ -15,6 +15,10 @@ length of the sequence at hand, so a position's encoding is the same however the
 YaRN (Peng, Quesnelle, Fan, Shippole: "YaRN: Efficient Context Window Extension of Large Language Models") divides by `factor`
 the frequencies that turn fewer than `slow` times over the original length, keeps those that turn more than `fast` times,
 blends linearly between, and multiplies cosine and sine by 0.1 ln(factor) + 1.
+
+"llama3" (the scaling of Llama 3.1's rotary frequencies) also divides the slow ones by `factor` - those that turn fewer than `low`
+times over the original length - and keeps those that turn more than `high` times; between, the two are blended linearly in the
+number of turns, and cosine and sine stay as they are.
 """
 from __future__ import annotations
 
@@ -104,6 +108,31 @@ class YarnRope(Rope):
         self.mscale = 0.1 * math.log(factor) + 1.0
 
 
+def llama3_inv_freq(rot_dim: int, theta: float, factor: float, original: float, low: float, high: float) -> List[float]:
+    out = []
+    for f in rotary_inv_freq(rot_dim, theta, None):
+        turns = original * f / (2.0 * math.pi)
+        if turns < low:
+            f = f / factor
+        elif turns <= high:
+            keep = (turns - low) / (high - low)
+            f = (1.0 - keep) * f / factor + keep * f
+        out.append(f)
+    return out
+
+
+class Llama3Rope(Rope):
+    """params: rot_dim, theta, interleaved, factor, original (positions), low, high (turns over them)."""
+
+    def __init__(self, params, prefix, dtype):
+        super().__init__(params, prefix, dtype)
+        factor, original = float(params["factor"]), float(params["original"])
+        low, high = float(params["low"]), float(params["high"])
+        if min(factor, original) <= 0.0 or not low < high:
+            raise ValueError("llama3: factor and original must be positive, low below high")
+        self._table = llama3_inv_freq(self.rot_dim, self.theta, factor, original, low, high)
+
+
 class NoPosition(PositionEncoding):
     """No position encoding (rot_dim 0)."""
 
@@ -115,4 +144,5 @@ class NoPosition(PositionEncoding):
 register_part("position", "rope", Rope)
 register_part("position", "longrope", LongRope)
 register_part("position", "yarn", YarnRope)
+register_part("position", "llama3", Llama3Rope)
 register_part("position", "none", NoPosition)

@@ -24,7 +24,7 @@ class LayerSpec:
     arrangement: str                            # registry key of the block, e.g. "prenorm_residual"
     mixer_norm: PartSpec
     mixer: PartSpec
-    ffn_norm: Optional[PartSpec]                # None (with ffn None): the layer has no feed-forward
+    ffn_norm: Optional[PartSpec]                # None: the layer has no feed-forward, or one that reads the mixer's norm (`one_norm`)
     ffn: Optional[PartSpec]
     params: Dict[str, Any] = field(default_factory=dict)   # e.g. {"residual_scale": s}
 
@@ -52,6 +52,7 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     pass_vectors: Optional[PartSpec] = None     # a table of residual-wide vectors that `RunStep.add_row` names
+    token_table: Optional[PartSpec] = None      # a table with a row per token that every layer takes its own columns of
 
 
 @dataclass
@@ -70,6 +71,7 @@ class WeightSpec:
     init: Tuple = ("normal", 0.02)
     fallback: Optional[str] = None
     free: Optional[int] = None
+    optional: bool = False                      # the checkpoint may lack it: the part is then not given it (random weights have none)
 
     def fits(self, shape) -> bool:
         shape = tuple(shape)

@@ -118,7 +118,8 @@ def check_against(model, source: TensorSource) -> None:
                 if not ws.fits(shape):
                     wrong.append((f"{full} (taken from {full_fb})", tuple(shape), tuple(ws.shape)))
                 continue
-            missing.append(full)
+            if not ws.optional:
+                missing.append(full)
             continue
         dt, shape = source.info(full)
         if not ws.fits(shape):
@@ -144,6 +145,8 @@ def load_into(model, source: TensorSource, device: torch.device,
         for ws in part.weight_specs():
             full = part.full_name(ws.name)
             src_name = full if full in have else ws.fallback
+            if src_name is None and ws.optional:
+                continue
             if src_name in shared:
                 tensors[ws.name] = shared[src_name]
                 continue

@@ -39,7 +39,7 @@ def random_tensors(cfg: ModelConfig, seed: int, device: str = "cpu", dtype: Opti
     out: Dict[str, torch.Tensor] = {}
     for part, ws in model.weight_specs():
         full = part.full_name(ws.name)
-        if ws.fallback is not None and tie:
+        if (ws.fallback is not None and tie) or ws.optional:
             continue
         g = torch.Generator(device=dev)
         g.manual_seed(_seed_for(seed, full))
