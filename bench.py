@@ -175,7 +175,7 @@ def timeline_step(args) -> int:
     raw = dict(CONFIG_05B if args.sizes == "0.5b" else CONFIG_8B)
     raw["num_hidden_layers"] = args.layers or 4
     if args.design != "default":                  # one of the pair of `--workload designs`, at the first of --design-sizes
-        pair = {"gopitar": gopitar_pair, "somipel": somipel_pair, "zokuzen": zokuzen_pair, "zibinex": zibinex_pair}.get(args.design, design_pair)
+        pair = {"gopitar": gopitar_pair, "somipel": somipel_pair, "zokuzen": zokuzen_pair, "zibinex": zibinex_pair, "gukosun": gukosun_pair}.get(args.design, design_pair)
         raw = pair(args.design_sizes.split(",")[0], args.layers or 4)[1 if args.design == "dense" else 0]
         raw["num_hidden_layers"] = args.layers or 4
     cfg = config_from_json(raw)
@@ -386,6 +386,24 @@ def zibinex_pair(size: str, layers: int):
     return zb, nz
 
 
+def gukosun_pair(size: str, layers: int):
+    """(Gukosun configuration, Gopitar configuration of the same width, depth, heads, head size, vocabulary and feed-forward width:
+    the framework's other design that mixes by softmax attention beside a decayed linear attention.) Even layers mix by attention
+    over a window of 1,024 with blended values, odd ones by capped attention over all positions beside linear attention; 2 kv
+    heads; every layer has a token input of 256 columns. (Gopitar's feed-forward is gated, three matrices of that width to two here.)"""
+    gp = gopitar_pair(size, layers)[0]
+    W, m, ff = gp["width"], gp["layers"][0]["mixer"], gp["layers"][0]["mlp"]["ff"]
+    H, d = m["left"]["heads"], m["left"]["dim"]
+    mlp = {"kind": "dense", "ff": ff}
+    att = {"heads": H, "kv_heads": 2, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": 1024}, "v_mix": True}
+    left = {"heads": H, "kv_heads": 2, "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 20.0,
+            "rot": {"base": 10000.0, "dims": d, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    par = {"left": left, "right": dict(m["right"])}
+    gk = {"architecture": "Gukosun", "vocab": gp["vocab"], "width": W, "norm": {"eps": 1e-5}, "logit_scale": 1.0, "token_side": {"dim": 256},
+          "layers": [{"type": "parallel", "mixer": par, "mlp": mlp} if i % 2 else {"type": "attention", "mixer": att, "mlp": mlp} for i in range(layers)]}
+    return gk, gp
+
+
 class OpTimer:
     """Brackets every kernel wrapper of `infinilm_b200.ops`, every library product of `Linear` and the library's grouped
     product with CUDA events on the launching stream, for steps that run eagerly; `table()` gives microseconds and calls per name."""
@@ -429,7 +447,8 @@ class OpTimer:
                      "gemm_tc5", "latent_norm_store", "moe_route", "moe_sort", "moe_combine", "gather_rows", "gemm_grouped", "short_conv",
                      "short_conv_state", "delta_prep", "matrix_state_scan", "group_norm_gate", "head_gate", "scaled_sum", "softcap", "silu_cols", "norm_add", "cast_rows",
                      "qk_norm_store", "gate_pack", "stabilized_gates", "hyper_step", "qk_rows_norm_rope_store", "token_shift_mix",
-                     "double_exp_decay", "tanh_rows", "moe_select", "moe_route_sort_small", "norm_add_norm", "latent_rope_store"):
+                     "double_exp_decay", "tanh_rows", "moe_select", "moe_route_sort_small", "norm_add_norm", "latent_rope_store", "branch_sum", "relu2",
+                     "gelu_row", "gemm_skinny_gelu_row"):
             self._wrap(ops, name)
         self._wrap(Linear, "__call__", "linear")
         if hasattr(F, "grouped_mm"):
@@ -468,8 +487,8 @@ def run_designs(args) -> int:
         rec = {"workload": "designs", "size": size, "layers": L, "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src}}
         family = getattr(args, "design_family", "nirozen")
         rec["design"] = family
-        pair = {"gopitar": gopitar_pair, "somipel": somipel_pair, "zokuzen": zokuzen_pair, "zibinex": zibinex_pair}.get(family, design_pair)
-        for which, raw in zip((family, {"somipel": "gopitar", "zokuzen": "nirozen", "zibinex": "nirozen"}.get(family, "dense_gqa")), pair(size, L)):
+        pair = {"gopitar": gopitar_pair, "somipel": somipel_pair, "zokuzen": zokuzen_pair, "zibinex": zibinex_pair, "gukosun": gukosun_pair}.get(family, design_pair)
+        for which, raw in zip((family, {"somipel": "gopitar", "zokuzen": "nirozen", "zibinex": "nirozen", "gukosun": "gopitar"}.get(family, "dense_gqa")), pair(size, L)):
             cfg = config_from_json(raw)
             B = 64
             eng = Engine.from_tensors(cfg, random_tensors(cfg, 0, "cuda:0"), dtype="bfloat16", page_size=PAGE,
@@ -570,11 +589,11 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 and 64 points")
     ap.add_argument("--no-graph", action="store_true", help="do not replay decode steps as CUDA graphs")
     ap.add_argument("--points", type=str, default="1,64", help="batch sizes of the extra decode points")
-    ap.add_argument("--design", choices=["default", "nirozen", "gopitar", "somipel", "zokuzen", "zibinex", "dense"], default="default",
+    ap.add_argument("--design", choices=["default", "nirozen", "gopitar", "somipel", "zokuzen", "zibinex", "gukosun", "dense"], default="default",
                     help="--timeline: the step of one of the pair of --workload designs instead of the benchmark model")
-    ap.add_argument("--design-family", choices=["nirozen", "gopitar", "somipel", "zokuzen", "zibinex"], default="nirozen",
+    ap.add_argument("--design-family", choices=["nirozen", "gopitar", "somipel", "zokuzen", "zibinex", "gukosun"], default="nirozen",
                     help="--workload designs: which design stands beside the dense GQA model of equal size (somipel: beside gopitar; "
-                         "zokuzen, zibinex: beside nirozen)")
+                         "gukosun: beside gopitar; zokuzen, zibinex: beside nirozen)")
     ap.add_argument("--design-sizes", type=str, default="1k,2k", help="--workload designs: layer sizes to run (1k, 2k, 4k)")
     ap.add_argument("--workload", choices=["default", "long_context", "continuous", "designs"], default="default",
                     help="default: the benchmark line. long_context: 8 requests x 16,384-token prompts at 8B sizes, prompt "

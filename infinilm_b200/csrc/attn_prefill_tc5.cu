@@ -35,7 +35,8 @@
 //   LOGB (with SIG): the bias by distance is pb_h - r1_h ln(1 + r2_h n), made here of three numbers per head instead of read
 //   from a table: a logarithm more per score, no loads (64 a row and tile) and no registers for them.
 //
-//   CAP: softmax over soft-capped scores, cap * tanh(scaled score / cap).
+//   CAP: softmax over soft-capped scores, cap * tanh(scaled score / cap): where a warp's scores of a tile lie well below the cap by a
+//   polynomial, else by an exponential and half a reciprocal a score.
 //
 //   Pages past the entry's last page are read as the last page again (finite values the mask removes).
 //   Every mbarrier wait is bounded; one that runs out sets *status and all roles leave their loops.
@@ -297,6 +298,8 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
         const float lb_pb = LOGB ? log_bias[2 * nh + g * G + hh] * 1.4426950408889634f : 0.f;
         const float* db_row = dist_bias ? dist_bias + g * G + hh : nullptr;
         const float db_far = dist_bias ? db_row[(size_t)dist_far * nh] * inv_scale : 0.f;
+        const float cap_kx = k_scale * 0.34657359027997264f;      // (ln 2 / 2)
+        const IlCapPoly poly = il_cap_poly(cap_kx, cap_log2);
         for (int j = 0; j < n_tiles; ++j) {
             const int b = j & 1;
             if (!t5_mbar_wait(s_full0 + 8 * b, (uint32_t)(j >> 1) & 1u, PT_SPIN)) { atomicExch(status, 36); ok = false; break; }
@@ -324,14 +327,29 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
                         sv[c] = __float_as_uint(fmaf(db_row[max(0, min(rpos - kb - c, dist_far)) * nh], inv_scale, __uint_as_float(sv[c])));
                 }
             }
-            if constexpr (CAP) {                  // cap * tanh(score / cap) as 1 - 2 / (1 + 2^(k s)), one reciprocal for two scores
+            if constexpr (CAP) {
+                float am[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                for (int c = 0; c < PT_KEYS; c += 2) {
-                    const float a = 1.f + pt_ex2(fminf(__uint_as_float(sv[c]) * k_scale, 60.f));
-                    const float bb = 1.f + pt_ex2(fminf(__uint_as_float(sv[c + 1]) * k_scale, 60.f));
-                    const float rr = __fdividef(-2.f * cap_log2, a * bb);
-                    sv[c] = __float_as_uint(fmaf(rr, bb, cap_log2));
-                    sv[c + 1] = __float_as_uint(fmaf(rr, a, cap_log2));
+                for (int c = 0; c < PT_KEYS; c += 4)
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) am[i] = fmaxf(am[i], fabsf(__uint_as_float(sv[c + i])));
+                if (!__any_sync(0xffffffffu, !(fmaxf(fmaxf(am[0], am[1]), fmaxf(am[2], am[3])) * cap_kx <= IL_CAP_SMALL))) {
+                    // far below the cap, as most scores are: a polynomial, so that the special-function unit has the softmax to itself
+#pragma unroll
+                    for (int c = 0; c < PT_KEYS; c += 2) {
+                        float a, bb;
+                        il_f2_get(il_cap_log2_small(il_f2_make(__uint_as_float(sv[c]), __uint_as_float(sv[c + 1])), poly), a, bb);
+                        sv[c] = __float_as_uint(a), sv[c + 1] = __float_as_uint(bb);
+                    }
+                } else {                          // cap * tanh(score / cap) as 1 - 2 / (1 + 2^(k s)), one reciprocal for two scores
+#pragma unroll
+                    for (int c = 0; c < PT_KEYS; c += 2) {
+                        const float a = 1.f + pt_ex2(fminf(__uint_as_float(sv[c]) * k_scale, 60.f));
+                        const float bb = 1.f + pt_ex2(fminf(__uint_as_float(sv[c + 1]) * k_scale, 60.f));
+                        const float rr = __fdividef(-2.f * cap_log2, a * bb);
+                        sv[c] = __float_as_uint(fmaf(rr, bb, cap_log2));
+                        sv[c + 1] = __float_as_uint(fmaf(rr, a, cap_log2));
+                    }
                 }
             }
             if (kb + PT_KEYS - 1 > rpos || kb < rlo) {        // the tile touches this row's causal or window edge
@@ -370,12 +388,26 @@ __global__ void __launch_bounds__(PT_THREADS, PT_BLOCKS_PER_SM) attn_prefill_tc5
                 corr = raise ? pt_ex2(m - m_new) : 1.f;   // 0 when nothing was summed yet
                 const float msafe = (m_new == -INFINITY) ? 0.f : m_new;
                 float sum4[4] = {0.f, 0.f, 0.f, 0.f};
+                if constexpr (CAP) {              // (the capped scores are in base 2 already; two at a time)
+                    const il_f2 neg_m = il_f2_dup(-msafe);
+                    il_f2 acc[2] = {il_f2_dup(0.f), il_f2_dup(0.f)};
 #pragma unroll
-                for (int c = 0; c < PT_KEYS; c += 2) {
-                    const float a = pt_ex2(fmaf(__uint_as_float(sv[c]), scale_log2, -msafe));
-                    const float bb = pt_ex2(fmaf(__uint_as_float(sv[c + 1]), scale_log2, -msafe));
-                    sum4[(c >> 1) & 3] += a + bb;
-                    sv[c >> 1] = pt_pack(a, bb);
+                    for (int c = 0; c < PT_KEYS; c += 2) {
+                        float a, bb;
+                        il_f2_get(il_f2_add(il_f2_make(__uint_as_float(sv[c]), __uint_as_float(sv[c + 1])), neg_m), a, bb);
+                        a = pt_ex2(a), bb = pt_ex2(bb);
+                        acc[(c >> 1) & 1] = il_f2_add(acc[(c >> 1) & 1], il_f2_make(a, bb));
+                        sv[c >> 1] = pt_pack(a, bb);
+                    }
+                    il_f2_get(acc[0], sum4[0], sum4[1]), il_f2_get(acc[1], sum4[2], sum4[3]);
+                } else {
+#pragma unroll
+                    for (int c = 0; c < PT_KEYS; c += 2) {
+                        const float a = pt_ex2(fmaf(__uint_as_float(sv[c]), scale_log2, -msafe));
+                        const float bb = pt_ex2(fmaf(__uint_as_float(sv[c + 1]), scale_log2, -msafe));
+                        sum4[(c >> 1) & 3] += a + bb;
+                        sv[c >> 1] = pt_pack(a, bb);
+                    }
                 }
                 l = l * corr + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
                 m = m_new;

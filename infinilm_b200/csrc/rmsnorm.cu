@@ -460,17 +460,20 @@ static int bs_launch(float* resid, const BsTerms& ts, void* copy, const void* wn
     return IL_OK;
 }
 
-// The branches come as parallel arrays of n_terms entries on the host.
-IL_EXPORT int il_branch_sum(float* resid, const void* const* y, const void* const* nw, const int* nw_kind, const void* const* cs, const int* cs_kind,
-                            const float* scale, const float* eps, int n_terms, void* copy, const void* wn, int wn_kind, float eps_n, void* out,
+// Branches behind the n_terms-th are not looked at. kinds: bit i: nw_i is bfloat16 (else f32), bit 8 + i: cs_i is.
+IL_EXPORT int il_branch_sum(float* resid, int n_terms, const void* y0, const void* y1, const void* y2, const void* y3, const void* nw0, const void* nw1,
+                            const void* nw2, const void* nw3, const void* cs0, const void* cs1, const void* cs2, const void* cs3, int kinds, float s0, float s1,
+                            float s2, float s3, float e0, float e1, float e2, float e3, void* copy, const void* wn, int wn_kind, float eps_n, void* out,
                             int act_kind, int n_rows, int H, cudaStream_t stream) {
     if (n_rows <= 0) return IL_OK;
     if (n_terms <= 0 || n_terms > BS_MAX_TERMS || H <= 0 || (!resid && !copy) || (out && (!wn || !resid))) return IL_BAD_ARG;
     if (act_kind != IL_F32 && act_kind != IL_BF16) return IL_BAD_ARG;
+    const void *y[] = {y0, y1, y2, y3}, *nw[] = {nw0, nw1, nw2, nw3}, *cs[] = {cs0, cs1, cs2, cs3};
+    const float scale[] = {s0, s1, s2, s3}, eps[] = {e0, e1, e2, e3};
     BsTerms ts = {};
     for (int i = 0; i < n_terms; ++i) {
         if (!y[i]) return IL_BAD_ARG;
-        ts.t[i] = BsTerm{y[i], nw[i], cs[i], nw_kind[i], cs_kind[i], scale[i], eps[i]};
+        ts.t[i] = BsTerm{y[i], nw[i], cs[i], (kinds >> i) & 1 ? IL_BF16 : IL_F32, (kinds >> (8 + i)) & 1 ? IL_BF16 : IL_F32, scale[i], eps[i]};
     }
     int rc = IL_OK;
 #define BS_PICK(TA)                                                                                           \

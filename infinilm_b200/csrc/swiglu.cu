@@ -71,9 +71,9 @@ __global__ void relu2_kernel(const TA* z, TA* out, size_t total_vec) {
     }
 }
 
-// out[t, n] = gelu_tanh(z[t, n]) * table[ids[t], off + n] for n < dim, 0 for dim <= n < ldo: a token's own row of a table, gated.
+// out[t, n] = gelu_tanh(z[t, n]) * table[ids[t], off + n] for n < dim, 0 for dim <= n < ldo: a token's own row of a table, gated (z f32).
 template <typename TA>
-__global__ void gelu_row_kernel(const TA* z, int ldz, const int* __restrict__ ids, const TA* __restrict__ table, int ldt, int off, int dim, int vocab,
+__global__ void gelu_row_kernel(const float* z, int ldz, const int* __restrict__ ids, const TA* __restrict__ table, int ldt, int off, int dim, int vocab,
                                 TA* __restrict__ out, int ldo, long long total) {
     il_pdl_wait();
     const long long stride = (long long)gridDim.x * blockDim.x;
@@ -82,7 +82,7 @@ __global__ void gelu_row_kernel(const TA* z, int ldz, const int* __restrict__ id
         const int n = (int)(i - t * ldo), id = ids[t];
         float y = 0.f;
         if (n < dim && id >= 0 && id < vocab) {   // (the host rejects other ids before launch; never read out of range)
-            const float g = il_to_f(z[t * ldz + n]), e = il_to_f(table[(size_t)id * ldt + off + n]);
+            const float g = z[t * ldz + n], e = il_to_f(table[(size_t)id * ldt + off + n]);
             y = sizeof(TA) == 2 ? il_gelu_tanh_mul_fast(g, e) : il_gelu_tanh_mul(g, e);
         }
         out[i] = il_from_f<TA>(y);
@@ -171,16 +171,16 @@ IL_EXPORT int il_relu2(const void* z, void* out, int act_kind, long long total, 
     return IL_OK;
 }
 
-IL_EXPORT int il_gelu_row(const void* z, int act_kind, int ldz, const int* ids, const void* table, int ldt, int off, int dim, int vocab, void* out,
+IL_EXPORT int il_gelu_row(const float* z, int act_kind, int ldz, const int* ids, const void* table, int ldt, int off, int dim, int vocab, void* out,
                           int ldo, int T, cudaStream_t stream) {
     if (T <= 0) return IL_OK;
     if (dim <= 0 || ldz < dim || ldo < dim || off < 0 || off + dim > ldt || vocab <= 0) return IL_BAD_ARG;
     const long long total = (long long)T * ldo, g = (total + 255) / 256;
     const int blocks = (int)(g > 148 * 16 ? 148 * 16 : g);
     if (act_kind == IL_F32)
-        IL_LAUNCH(gelu_row_kernel<float>, blocks, 256, 0, stream, (const float*)z, ldz, ids, (const float*)table, ldt, off, dim, vocab, (float*)out, ldo, total);
+        IL_LAUNCH(gelu_row_kernel<float>, blocks, 256, 0, stream, z, ldz, ids, (const float*)table, ldt, off, dim, vocab, (float*)out, ldo, total);
     else if (act_kind == IL_BF16)
-        IL_LAUNCH(gelu_row_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (const __nv_bfloat16*)z, ldz, ids, (const __nv_bfloat16*)table, ldt, off, dim, vocab,
+        IL_LAUNCH(gelu_row_kernel<__nv_bfloat16>, blocks, 256, 0, stream, z, ldz, ids, (const __nv_bfloat16*)table, ldt, off, dim, vocab,
                   (__nv_bfloat16*)out, ldo, total);
     else
         return IL_BAD_ARG;

@@ -200,15 +200,16 @@ def _check_row_table(name: str, ids: torch.Tensor, table: torch.Tensor, off: int
 
 
 def gelu_row(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, off: int, dim: int, out: torch.Tensor) -> None:
-    """out[t, n] = gelu_tanh(z[t, n]) * table[ids[t], off + n] for n < dim, 0 in out's columns behind them."""
+    """out[t, n] = gelu_tanh(z[t, n]) * table[ids[t], off + n] for n < dim, 0 in out's columns behind them; z float32, out and table of
+    one dtype."""
     _need_cuda(z, ids, table, out)
     T = z.shape[0]
-    _check_row_table("gelu_row", ids, table, off, dim, T, z.dtype)
-    if z.stride(1) != 1 or z.shape[1] < dim or out.dtype != z.dtype or out.shape[0] != T or out.shape[1] < dim or not out.is_contiguous():
-        raise KernelError("gelu_row: z [T, >= dim], out [T, >= dim] contiguous, one dtype")
+    _check_row_table("gelu_row", ids, table, off, dim, T, out.dtype)
+    if z.dtype != torch.float32 or z.stride(1) != 1 or z.shape[1] < dim or out.shape[0] != T or out.shape[1] < dim or not out.is_contiguous():
+        raise KernelError("gelu_row: z float32 [T, >= dim], out [T, >= dim] contiguous")
     f = _fn("swiglu", "il_gelu_row", [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int,
                                       _c_void_p])
-    _check(f(_ptr(z), kind_of(z.dtype), z.stride(0), _ptr(ids), _ptr(table), table.stride(0), off, dim, table.shape[0], _ptr(out), out.shape[1], T,
+    _check(f(_ptr(z), kind_of(out.dtype), z.stride(0), _ptr(ids), _ptr(table), table.stride(0), off, dim, table.shape[0], _ptr(out), out.shape[1], T,
              _stream()), "gelu_row")
 
 
@@ -408,15 +409,19 @@ def branch_sum(terms, resid: Optional[torch.Tensor] = None, copy: Optional[torch
             raise KernelError("branch_sum: copy and out [T,H] of the branches' dtype")
     if next_weight is not None and (next_weight.numel() != H or not next_weight.is_contiguous()):
         raise KernelError("branch_sum: next_weight [H]")
-    vp, ci, cf = _c_void_p * n, _c_int * n, _c_float * n
-
-    def kinds(name):
-        return ci(*[0 if getattr(t, name) is None else kind_of(getattr(t, name).dtype) for t in terms])
-    f = _fn("rmsnorm", "il_branch_sum", [_c_void_p] * 8 + [_c_int, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_void_p])
-    _check(f(_ptr(resid), vp(*[t.y.data_ptr() for t in terms]), vp(*[_ptr(t.norm_weight) for t in terms]), kinds("norm_weight"),
-             vp(*[_ptr(t.col_scale) for t in terms]), kinds("col_scale"), cf(*[t.scale for t in terms]), cf(*[t.eps for t in terms]), n,
-             _ptr(copy), _ptr(next_weight if out is not None else None), kind_of(next_weight.dtype) if out is not None else 0, next_eps, _ptr(out),
-             kind_of(dt), T, H, _stream()), "branch_sum")
+    ys, nws, css, ss, es, kinds = [0] * 4, [0] * 4, [0] * 4, [0.0] * 4, [0.0] * 4, 0
+    for i, t in enumerate(terms):
+        ys[i], ss[i], es[i] = t.y.data_ptr(), t.scale, t.eps
+        if t.norm_weight is not None:
+            nws[i] = t.norm_weight.data_ptr()
+            kinds |= kind_of(t.norm_weight.dtype) << i
+        if t.col_scale is not None:
+            css[i] = t.col_scale.data_ptr()
+            kinds |= kind_of(t.col_scale.dtype) << (8 + i)
+    f = _fn("rmsnorm", "il_branch_sum", [_c_void_p, _c_int] + [_c_void_p] * 12 + [_c_int] + [_c_float] * 8
+            + [_c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_void_p])
+    _check(f(_ptr(resid), n, *ys, *nws, *css, kinds, *ss, *es, _ptr(copy), _ptr(next_weight if out is not None else None),
+             kind_of(next_weight.dtype) if out is not None else 0, next_eps, _ptr(out), kind_of(dt), T, H, _stream()), "branch_sum")
 
 
 HYPER_MAX_STREAMS = 16

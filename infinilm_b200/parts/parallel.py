@@ -42,6 +42,8 @@ class ParallelMixers(Mixer):
         self.norm_w: Dict[str, torch.Tensor] = {}
         if self.norm_eps is not None and len(self.branches) > ops.BRANCH_MAX_TERMS:
             raise ValueError(f"parallel mixers: at most {ops.BRANCH_MAX_TERMS} normed branches")
+        kinds = [spec.kind for spec, _ in params["branches"]]
+        self._kind_again = [k in kinds[i + 1:] for i, k in enumerate(kinds)]       # a later branch writes its output where this one's lies
         self._n_needs = [len(_needs_of(m)) for m in self.branches]
         self._single = [not isinstance(m.cache_need(), (tuple, list)) for m in self.branches]
 
@@ -76,14 +78,17 @@ class ParallelMixers(Mixer):
     def forward(self, x, ctx, cache, tail=None, terms=False):
         views = list(cache) if isinstance(cache, (tuple, list)) else ([] if cache is None else [cache])
         at, ys = 0, []
-        for m, n, single, scale in zip(self.branches, self._n_needs, self._single, self.scales):
+        for m, n, single, scale, again in zip(self.branches, self._n_needs, self._single, self.scales, self._kind_again):
             mine = views[at: at + n]
             at += n
             mine = (mine[0] if mine else None) if single else tuple(mine)
             if tail is not None:
                 ys.append(m.forward(x, ctx, mine, tail=ResidualTail(tail.resid, tail.scale * scale, tail.norm)))
             else:
-                ys.append(m.forward(x, ctx, mine))
+                y = m.forward(x, ctx, mine)
+                if again:
+                    y = ctx.ws.rows(f"parallel_out{len(ys)}", y.shape[0], y.shape[1], y.dtype).copy_(y)
+                ys.append(y)
         if tail is not None:
             return ys[-1]
         if terms or self.norm_eps is not None:

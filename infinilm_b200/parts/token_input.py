@@ -49,6 +49,6 @@ class TokenInput(Part):
         if self.dtype == torch.bfloat16 and ops.skinny_ok(T, self.hidden):
             ops.gemm_skinny_gelu_row(x, self.gate.weight, ctx.token_ids, table, self.offset, self.dim, g)
         else:
-            z = self.gate(x, ctx.ws.rows("token_gate", T, self.dim_pad, self.dtype))
+            z = self.gate(x, ctx.ws.rows("token_gate", T, self.dim_pad, torch.float32), out_f32=True)
             ops.gelu_row(z, ctx.token_ids, table, self.offset, self.dim, g)
         return self.proj(g, ctx.ws.rows("token_branch", T, self.hidden, self.dtype))

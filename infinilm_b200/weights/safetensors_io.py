@@ -111,7 +111,7 @@ def write_safetensors(path: str, tensors: Dict[str, torch.Tensor], metadata: Opt
         f.write(hj)
         for name in order:
             t = tensors[name].detach().contiguous().cpu()
-            f.write(t.view(torch.uint8).reshape(-1).numpy().tobytes() if t.numel() else b"")
+            f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")
     os.replace(tmp, path)
 
 
