@@ -74,18 +74,50 @@ __global__ void relu2_kernel(const TA* z, TA* out, size_t total_vec) {
 // out[t, n] = gelu_tanh(z[t, n]) * table[ids[t], off + n] for n < dim, 0 for dim <= n < ldo: a token's own row of a table, gated (z f32).
 template <typename TA>
 __global__ void gelu_row_kernel(const float* z, int ldz, const int* __restrict__ ids, const TA* __restrict__ table, int ldt, int off, int dim, int vocab,
-                                TA* __restrict__ out, int ldo, long long total) {
+                                TA* __restrict__ out, int ldo, unsigned total) {
     il_pdl_wait();
-    const long long stride = (long long)gridDim.x * blockDim.x;
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
-        const long long t = i / ldo;
-        const int n = (int)(i - t * ldo), id = ids[t];
+    const unsigned stride = gridDim.x * blockDim.x;
+    for (unsigned i = blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
+        const unsigned t = i / (unsigned)ldo;
+        const int n = (int)(i - t * (unsigned)ldo), id = ids[t];
         float y = 0.f;
         if (n < dim && id >= 0 && id < vocab) {   // (the host rejects other ids before launch; never read out of range)
-            const float g = z[t * ldz + n], e = il_to_f(table[(size_t)id * ldt + off + n]);
+            const float g = z[(size_t)t * ldz + n], e = il_to_f(table[(size_t)id * ldt + off + n]);
             y = sizeof(TA) == 2 ? il_gelu_tanh_mul_fast(g, e) : il_gelu_tanh_mul(g, e);
         }
         out[i] = il_from_f<TA>(y);
+    }
+}
+
+// The same, four neighbouring columns a thread.
+__device__ __forceinline__ float4 gr_ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 gr_ld4(const __nv_bfloat16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void gr_st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void gr_st4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+template <typename TA>
+__global__ void gelu_row4_kernel(const float* z, int ldz, const int* __restrict__ ids, const TA* __restrict__ table, int ldt, int off, int dim, int vocab,
+                                 TA* __restrict__ out, int ldo, unsigned total4) {
+    il_pdl_wait();
+    const unsigned stride = gridDim.x * blockDim.x, ld4 = (unsigned)ldo >> 2;
+    for (unsigned i = blockIdx.x * blockDim.x + threadIdx.x; i < total4; i += stride) {
+        const unsigned t = i / ld4;
+        const int n = (int)(i - t * ld4) << 2, id = ids[t];
+        float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (n < dim && id >= 0 && id < vocab) {   // (dim is a multiple of 4 here)
+            const float4 g = gr_ld4(z + (size_t)t * ldz + n), e = gr_ld4(table + (size_t)id * ldt + off + n);
+            if (sizeof(TA) == 2)
+                y = make_float4(il_gelu_tanh_mul_fast(g.x, e.x), il_gelu_tanh_mul_fast(g.y, e.y), il_gelu_tanh_mul_fast(g.z, e.z), il_gelu_tanh_mul_fast(g.w, e.w));
+            else
+                y = make_float4(il_gelu_tanh_mul(g.x, e.x), il_gelu_tanh_mul(g.y, e.y), il_gelu_tanh_mul(g.z, e.z), il_gelu_tanh_mul(g.w, e.w));
+        }
+        gr_st4(out + (size_t)t * ldo + n, y);
     }
 }
 
@@ -175,15 +207,29 @@ IL_EXPORT int il_gelu_row(const float* z, int act_kind, int ldz, const int* ids,
                           int ldo, int T, cudaStream_t stream) {
     if (T <= 0) return IL_OK;
     if (dim <= 0 || ldz < dim || ldo < dim || off < 0 || off + dim > ldt || vocab <= 0) return IL_BAD_ARG;
-    const long long total = (long long)T * ldo, g = (total + 255) / 256;
+    if (act_kind != IL_F32 && act_kind != IL_BF16) return IL_BAD_ARG;
+    const int eb = act_kind == IL_F32 ? 4 : 2;    // four columns at a time where every row's pieces start on whole borders
+    const bool vec = ((ldz | ldo | ldt | off | dim) & 3) == 0 && ((uintptr_t)z & 15) == 0 && (((uintptr_t)table | (uintptr_t)out) & (4 * eb - 1)) == 0;
+    const long long all = (long long)T * ldo, g = (all + 255) / 256;
+    if (all > 0x7fffffffLL) return IL_UNSUPPORTED;
+    const unsigned total = (unsigned)all;
     const int blocks = (int)(g > 148 * 16 ? 148 * 16 : g);
+    if (vec) {
+        const long long g4 = (all / 4 + 255) / 256;
+        const int blocks4 = (int)(g4 > 148 * 16 ? 148 * 16 : g4);
+        if (act_kind == IL_F32)
+            IL_LAUNCH(gelu_row4_kernel<float>, blocks4, 256, 0, stream, z, ldz, ids, (const float*)table, ldt, off, dim, vocab, (float*)out, ldo, total / 4);
+        else
+            IL_LAUNCH(gelu_row4_kernel<__nv_bfloat16>, blocks4, 256, 0, stream, z, ldz, ids, (const __nv_bfloat16*)table, ldt, off, dim, vocab,
+                      (__nv_bfloat16*)out, ldo, total / 4);
+        IL_LAUNCH_CHECK();
+        return IL_OK;
+    }
     if (act_kind == IL_F32)
         IL_LAUNCH(gelu_row_kernel<float>, blocks, 256, 0, stream, z, ldz, ids, (const float*)table, ldt, off, dim, vocab, (float*)out, ldo, total);
-    else if (act_kind == IL_BF16)
+    else
         IL_LAUNCH(gelu_row_kernel<__nv_bfloat16>, blocks, 256, 0, stream, z, ldz, ids, (const __nv_bfloat16*)table, ldt, off, dim, vocab,
                   (__nv_bfloat16*)out, ldo, total);
-    else
-        return IL_BAD_ARG;
     IL_LAUNCH_CHECK();
     return IL_OK;
 }
